@@ -21,6 +21,7 @@ GEMM_STORE_BF16 = 2
 GEMM_SWIGLU_BF16 = 3
 GEMM_RELU2_BF16 = 4
 GEMM_GLU_CLAMP_BF16 = 5
+GEMM_SOFTCAP_F32 = 6
 FLAG_PDL = 1
 FLAG_ORDERED = 2   # atx_gemm_run ADD_F32, T <= 64: fixed-order split-K (bit-reproducible)
 FLAG_ADD_BF16 = 4  # atx_rmsnorm: the `add` buffer is bf16
@@ -50,6 +51,7 @@ EXPORTS = [
     "atx_resid_norm_out", "atx_gated_act_clamped", "atx_gated_norm_groups", "atx_conv_residual", "atx_lowrank_logdecay",
     "atx_gated_linear_recurrence", "atx_moe_route_opts", "atx_gemm_plan_set_gate",
     "atx_gated_linear_recurrence_chunked", "atx_gated_linear_recurrence_chunked_supported",
+    "atx_parallel_resid_norm", "atx_conv_head_prepare", "atx_conv_dt_inplace", "atx_moe_route_scored", "atx_soft_cap",
 ]
 ATTN_SOFTMAX = 0
 ATTN_SIGMOID = 1
@@ -58,6 +60,11 @@ ACT_GELU_TANH = 1
 HEAD_DST_ROWS = 0
 HEAD_DST_PAGES = 1
 HEAD_SEGS_MAX = 4
+MOE_ACT_RELU2 = 2
+MOE_SOFTMAX = 0
+MOE_SIGMOID = 1
+TABLE_ADD = 1
+TABLE_START = 2
 
 
 class HeadSeg(C.Structure):
@@ -69,6 +76,22 @@ class HeadSeg(C.Structure):
                 ("mix", C.c_float), ("rot_half", C.c_int),
                 ("norm_w", C.c_void_p), ("rot", C.c_void_p), ("mix_src", C.c_void_p), ("save", C.c_void_p),
                 ("dst", C.c_void_p), ("dst_ld", C.c_longlong)]
+
+
+class ConvHeadSeg(C.Structure):
+    """atx_conv_head_seg: one slice of a projection row for atx_conv_head_prepare (include/atx_b200.h)."""
+
+    _fields_ = [("src_off", C.c_int), ("heads", C.c_int), ("width", C.c_int), ("norm", C.c_int), ("rot_dims", C.c_int),
+                ("dst_kind", C.c_int), ("w", C.c_void_p), ("rot", C.c_void_p), ("dst", C.c_void_p), ("raw_dst", C.c_void_p),
+                ("dst_ld", C.c_longlong)]
+
+
+class ResidTerms(C.Structure):
+    """atx_resid_terms: what atx_parallel_resid_norm adds to the stream (include/atx_b200.h)."""
+
+    _fields_ = [("y", C.c_void_p), ("experts", C.c_void_p), ("wgt", C.c_void_p), ("slot_of", C.c_void_p), ("ids", C.c_void_p),
+                ("table", C.c_void_p), ("vec", C.c_void_p), ("lde", C.c_longlong), ("y_scale", C.c_float),
+                ("zero_y", C.c_int), ("top", C.c_int), ("vocab", C.c_int), ("table_mode", C.c_int)]
 
 
 class AttnOpts(C.Structure):
@@ -83,6 +106,11 @@ class AttnOpts(C.Structure):
 def head_segs(*segs: "HeadSeg"):
     """A C array of segments for atx_head_prepare."""
     return (HeadSeg * len(segs))(*segs)
+
+
+def conv_head_segs(*segs: "ConvHeadSeg"):
+    """A C array of segments for atx_conv_head_prepare."""
+    return (ConvHeadSeg * len(segs))(*segs)
 
 
 class AtxError(RuntimeError):
@@ -207,6 +235,13 @@ def load() -> C.CDLL:
     lib.atx_gated_linear_recurrence_chunked.argtypes = list(lib.atx_gated_linear_recurrence.argtypes)
     lib.atx_gated_linear_recurrence_chunked_supported.argtypes = [i32]
     lib.atx_moe_route_opts.argtypes = [vp, i64, vp, i32, i32, f32, i32, vp, vp, i32, i32, vp]
+    lib.atx_parallel_resid_norm.argtypes = [vp, C.POINTER(ResidTerms), vp, vp, vp, vp, f32, vp, i32, i32, f32, vp, i64, i32, i32, vp]
+    lib.atx_conv_head_prepare.argtypes = [vp, i64, C.POINTER(ConvHeadSeg), i32, i32, vp, i32, i32, vp, vp, vp, vp, vp, vp, i32, i32,
+                                          f32, i32, i32, vp]
+    lib.atx_conv_dt_inplace.argtypes = [vp, i64, i32, i32, vp, vp, vp, vp, vp, vp, vp, vp, vp, vp, vp, vp, i32, i32, i32, i32, i32,
+                                        i32, i32, vp]
+    lib.atx_moe_route_scored.argtypes = [vp, i64, vp, i32, i32, f32, i32, i32, i32, vp, vp, i32, i32, vp]
+    lib.atx_soft_cap.argtypes = [vp, i64, i32, i32, f32, i32, vp]
     for name in EXPORTS:  # fail at load time, not at first use, if the build is stale
         getattr(lib, name)
     _lib = lib

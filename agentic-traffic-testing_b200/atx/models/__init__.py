@@ -10,9 +10,9 @@ from typing import Optional
 
 
 def _entries():
-    from . import gopopel, napuzen, safisun, zonidra
+    from . import gopopel, lifuzen, napuzen, safisun, zonidra
 
-    return {"safisun": safisun, "gopopel": gopopel, "zonidra": zonidra, "napuzen": napuzen}
+    return {"safisun": safisun, "gopopel": gopopel, "zonidra": zonidra, "napuzen": napuzen, "lifuzen": lifuzen}
 
 
 def _module(arch: str):

@@ -1,5 +1,5 @@
-"""What the layer programs of the layer-list families share: the linear layer that picks a GEMM kernel, and the table of
-rotation angles."""
+"""What the layer programs of the layer-list families share: the linear layer that picks a GEMM kernel, the table of
+rotation angles, the experts of a mixture without gates."""
 from __future__ import annotations
 
 import math
@@ -35,8 +35,8 @@ class _Linear:
             if zeroed and mode == _cabi.GEMM_STORE_F32 and self.accumulates(T):
                 rc = self.lib.atx_gemm_run(self.plan._h, out_ptr, ldo, T, _cabi.GEMM_ADD_F32, 0, flags, st)
             else:
-                rc = self.lib.atx_gemm_run(self.plan._h, out_ptr, ldo, T, mode, 1 if mode == _cabi.GEMM_STORE_F32 else 0,
-                                           flags, st)
+                whole_k = mode in (_cabi.GEMM_STORE_F32, _cabi.GEMM_SOFTCAP_F32)
+                rc = self.lib.atx_gemm_run(self.plan._h, out_ptr, ldo, T, mode, 1 if whole_k else 0, flags, st)
         else:
             assert mode in (_cabi.GEMM_STORE_F32, _cabi.GEMM_ADD_F32)
             rc = self.lib.atx_gemm_simple(self.w.data_ptr(), self.K, self.x.data_ptr(), self.K, out_ptr, ldo, T, self.N,
@@ -106,3 +106,70 @@ def rotation_table_scaled(freqs: List[float], magnitude: float, max_pos: int, de
     entries as they are, so a rotated pair comes out scaled)."""
     ang = torch.arange(max_pos, dtype=torch.float64)[:, None] * torch.tensor(freqs, dtype=torch.float64)[None, :]
     return (torch.cat((ang.cos(), ang.sin()), -1) * magnitude).to(torch.float32).contiguous().to(device)
+
+
+class UngatedExperts:
+    """The feed-forwards of a mixture of experts without gates, sum_k w_k W_down,e max(W_up,e x, 0)^2: routing, the plan that sorts
+    (token, choice) pairs by expert, the two products. The weighted sum is left to the kernel that consumes `out` by slot
+    (`slot_of`, `wgt`). One object serves every layer of a program (its buffers are reused from layer to layer)."""
+
+    def __init__(self, lib, ck, specs: List[dict], T: int, W: int, xn: torch.Tensor, dt: int):
+        """specs: the `mlp` entries of the model's layers (may be empty); xn [T, W]: the rows the experts read."""
+        dev, xt, i32 = xn.device, xn.dtype, torch.int32
+        self.lib, self.ck, self.W, self.dt, self.xn = lib, ck, W, dt, xn
+        top = max([int(m["router"]["top"]) for m in specs], default=1)
+        E = max([int(m["router"]["experts"]) for m in specs], default=1)
+        F = max([int(m["expert"]["ff"]) for m in specs], default=1)
+        P = T * top if specs else 1
+        self.P = P
+        self.sms = torch.cuda.get_device_properties(dev).multi_processor_count
+        self.tile_rows, self.big_rows = int(lib.atx_moe_tile_rows()), int(lib.atx_gemm_grouped_tile_rows())
+        self.max_tiles = max((P + self.tile_rows - 1) // self.tile_rows, (min(P, 64 * top) + 15) // 16) + E
+        self.max_big_tiles = (P + self.big_rows - 1) // self.big_rows + E
+        self.sel = torch.zeros(P, dtype=i32, device=dev)
+        self.wgt = torch.zeros(P, dtype=torch.float32, device=dev)
+        self.seg_off = torch.zeros(E + 1, dtype=i32, device=dev)
+        self.perm = torch.zeros(P, dtype=i32, device=dev)
+        self.slot_of = torch.zeros(P, dtype=i32, device=dev)
+        self.tiles = torch.zeros(2 + 2 * self.max_tiles, dtype=i32, device=dev)
+        self.tiles_big = torch.zeros(2 + 2 * self.max_big_tiles, dtype=i32, device=dev)
+        self.act = torch.zeros(P * F, dtype=xt, device=dev)
+        self.out = torch.zeros(P * W if specs else 1, dtype=torch.float32, device=dev)
+        self.grouped = any(_use_tc(xt, W) and int(m["expert"]["ff"]) % 64 == 0 for m in specs)
+        self.xperm = torch.zeros(P if self.grouped else 1, W, dtype=xt, device=dev)
+
+    def plans(self, w_up: torch.Tensor, w_down: torch.Tensor) -> Optional[dict]:
+        """GEMM plans of one layer for prompt-sized steps (w_up [E, F, W], w_down [E, W, F]), or None where the sizes have none."""
+        E, F, W = w_up.shape
+        if not (_use_tc(w_up.dtype, W) and F % 64 == 0):
+            return None
+        return {"up": _cabi.GemmPlan(w_up.view(E * F, W), self.xperm),
+                "down": _cabi.GemmPlan(w_down.view(E * W, F), self.act[:self.P * F].view(self.P, F))}
+
+    def run(self, logits: int, ld: int, top: int, w_up: torch.Tensor, w_down: torch.Tensor, plans: Optional[dict], T: int,
+            small: bool, fl: int, st: int) -> int:
+        """Router logits (device pointer, fp32 [T, ld]) -> sel, wgt (squared scores: the weight multiplies the input of an expert of
+        degree two), slot_of and `out` by slot. Returns the launch count."""
+        lib, ck, W, dt = self.lib, self.ck, self.W, self.dt
+        E, F = int(w_up.shape[0]), int(w_up.shape[1])
+        sel, so, pm, sl = (t.data_ptr() for t in (self.sel, self.seg_off, self.perm, self.slot_of))
+        pairs, act, out, x = T * top, self.act.data_ptr(), self.out.data_ptr(), self.xn.data_ptr()
+        ck(lib.atx_moe_route_scored(logits, ld, None, E, top, 1.0, 0, _cabi.MOE_SIGMOID, 2, sel, self.wgt.data_ptr(), T, fl, st))
+        if plans is not None and not small:
+            # prompt-sized: gather every expert's rows, then both products on the tcgen05 GEMM over the plan's tiles
+            big, tb = min(self.max_big_tiles, (pairs + self.big_rows - 1) // self.big_rows + E), self.tiles_big.data_ptr()
+            ck(lib.atx_moe_plan(sel, pairs, E, self.big_rows, so, pm, sl, tb, fl, st))
+            ck(lib.atx_moe_gather_rows(x, W, pm, top, so, E, self.xperm.data_ptr(), W, pairs, W, dt, fl, st))
+            ck(lib.atx_gemm_run_grouped(plans["up"]._h, act, F, F, _cabi.GEMM_RELU2_BF16, so, tb, big, fl, st))
+            ck(lib.atx_gemm_run_grouped(plans["down"]._h, out, W, W, _cabi.GEMM_STORE_F32, so, tb, big, fl, st))
+            return 5
+        # decode-sized bf16 steps (one or two rows per expert): tiles of 16 slots let more CTAs share an SM where two per SM
+        # would need a second wave
+        ctas = min(E, pairs) * ((F + 63) // 64)
+        tr = 16 if (small and dt == _cabi.DT_BF16 and ctas > 2 * self.sms) else self.tile_rows
+        tiles, tl = min(self.max_tiles, (pairs + tr - 1) // tr + E), self.tiles.data_ptr()
+        ck(lib.atx_moe_plan(sel, pairs, E, tr, so, pm, sl, tl, fl, st))
+        ck(lib.atx_moe_expert_gemm(x, W, pm, top, 1, w_up.data_ptr(), F * W, W, act, F, F, W, _cabi.MOE_ACT_RELU2, 0, tr, so, tl,
+                                   tiles, dt, fl, st))
+        ck(lib.atx_moe_expert_gemm(act, F, None, top, 0, w_down.data_ptr(), W * F, F, out, W, W, F, 0, 0, tr, so, tl, tiles, dt, fl, st))
+        return 4

@@ -26,6 +26,7 @@ namespace atx {
 
 // The gated epilogues: ATX_GEMM_SWIGLU_BF16 = silu(gate) * up; ATX_GEMM_GLU_CLAMP_BF16 = g sigmoid(alpha g) (u + shift) with
 // g = min(gate, limit), u = clamp(up, -limit, limit) (alpha, limit, shift: atx_gemm_plan_set_gate). Same tile layout.
+// ATX_GEMM_SOFTCAP_F32 = limit tanh(acc / limit), stored as fp32 (the cap on a model's logits).
 struct GateParams {
     float alpha, limit, shift;
 };
@@ -37,6 +38,9 @@ __device__ __forceinline__ float glu_value(float g, float u, int mode, const Gat
     g = fminf(g, gp.limit);
     u = fminf(fmaxf(u, -gp.limit), gp.limit);
     return g / (1.f + expf(-gp.alpha * g)) * (u + gp.shift);
+}
+__device__ __forceinline__ float stored_value(float a, int mode, const GateParams& gp) {
+    return mode == ATX_GEMM_SOFTCAP_F32 ? gp.limit * tanhf(a / gp.limit) : a;
 }
 
 
@@ -293,12 +297,12 @@ gemm_wt_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
             tmem_ld16(tmem_acc + (static_cast<uint32_t>(warp * 32) << 16) + c, v);
             tmem_ld_wait();
             if (n_ok) {
-                if (mode == ATX_GEMM_STORE_F32) {
+                if (mode == ATX_GEMM_STORE_F32 || mode == ATX_GEMM_SOFTCAP_F32) {
                     float* o = reinterpret_cast<float*>(out);
 #pragma unroll
                     for (int j = 0; j < 16; ++j) {
                         const int t = t0 + c + j;
-                        if (t < T) o[static_cast<long long>(t) * ldo + n] = __uint_as_float(v[j]);
+                        if (t < T) o[static_cast<long long>(t) * ldo + n] = stored_value(__uint_as_float(v[j]), mode, gate_params);
                     }
                 } else if (mode == ATX_GEMM_ADD_F32) {
                     // parked in shared memory (token-major) and added below, four consecutive outputs at a time
@@ -573,12 +577,13 @@ gemm_wt_persistent_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_
                     tmem_ld16(tlane + c, v);
                     tmem_ld_wait();
                     if (n_ok) {
-                        if (mode == ATX_GEMM_STORE_F32) {
+                        if (mode == ATX_GEMM_STORE_F32 || mode == ATX_GEMM_SOFTCAP_F32) {
                             float* o = reinterpret_cast<float*>(out);
 #pragma unroll
                             for (int j = 0; j < 16; ++j) {
                                 const int t = t0 + c + j;
-                                if (t < t_end) o[static_cast<long long>(t) * ldo + n] = __uint_as_float(v[j]);
+                                if (t < t_end)
+                                    o[static_cast<long long>(t) * ldo + n] = stored_value(__uint_as_float(v[j]), mode, gate_params);
                             }
                         } else if (mode == ATX_GEMM_ADD_F32) {
                             float* o = reinterpret_cast<float*>(out);
@@ -670,7 +675,7 @@ struct atx_gemm_plan {
     CUtensorMap tmX[5];  // one per token-tile size
     long long N, K, T_cap;
     int w_evict_first;
-    atx::GateParams gate;   // constants of ATX_GEMM_GLU_CLAMP_BF16
+    atx::GateParams gate;   // constants of ATX_GEMM_GLU_CLAMP_BF16 and ATX_GEMM_SOFTCAP_F32
 };
 
 using namespace atx;
@@ -850,7 +855,7 @@ int atx_gemm_run(const atx_gemm_plan* p, void* out, long long ldo, int T, int mo
     cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_);
     ATX_REQUIRE(p && out, "atx_gemm_run: null pointer");
     ATX_REQUIRE(T > 0 && T <= p->T_cap, "atx_gemm_run: T=%d outside (0, %lld]", T, p->T_cap);
-    ATX_REQUIRE(mode >= ATX_GEMM_STORE_F32 && mode <= ATX_GEMM_GLU_CLAMP_BF16, "atx_gemm_run: bad mode %d", mode);
+    ATX_REQUIRE(mode >= ATX_GEMM_STORE_F32 && mode <= ATX_GEMM_SOFTCAP_F32, "atx_gemm_run: bad mode %d", mode);
     ATX_REQUIRE(ldo >= (is_glu(mode) ? p->N / 2 : p->N), "atx_gemm_run: ldo=%lld too small for N=%lld", ldo, p->N);
     ATX_REQUIRE(!is_glu(mode) || p->N % 128 == 0, "atx_gemm_run: SWIGLU mode needs N %% 128 == 0");
     // ATX_FLAG_ORDERED: the K-splits of an ADD are reduced inside a cluster in a fixed order (as for SwiGLU) and ONE CTA

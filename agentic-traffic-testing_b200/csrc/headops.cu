@@ -6,6 +6,10 @@
 //     layer, and written either to a row buffer (queries, GEMM inputs) or into the paged cache at the token's slot.
 //     A launch takes up to four such slices, so that q, k and v of a layer (or the two bottlenecks of a latent
 //     attention) are prepared together,
+//   * the same for slices that first pass a short causal convolution over time, per channel, whose carried inputs live in
+//     the sequence's state slot; the convolved head can be kept as it is (values that are the keys) beside the rotated and
+//     normed one,
+//   * a cap on logits, c tanh(z / c), in place,
 //   * a small matrix product per head  out[t, h, :] = W_h x[t, h, :]  with an optional sigmoid gate per output element
 //     (the per-head up-projections of latent attention in its absorbed form).
 // Element type XT (weights, GEMM inputs, pages) = bf16 or fp32; sums, norms, rotations and blends are fp32.
@@ -282,6 +286,260 @@ head_prepare_kernel(const float* __restrict__ src, long long ld, const int* __re
     }
 }
 
+// ---- head preparation behind a short convolution ------------------------------------------------------------------------------
+// Per head of a slice: u_t = sum_j w[c][j] x_(t - K + 1 + j) per channel (no bias, no activation; zeros before position 0, the
+// K - 1 rows before the step from conv_state [slots, K - 1, C], channel = source column - the first slice's), u written to
+// raw_dst's pages as it is (nullable), pairs (2i, 2i + 1) of the first rot_dims elements rotated by the angles at the row's
+// position, divided by the root mean square over the head (norm != 0), written to rows or pages. Rows of sequences
+// [0, n_inplace) are the only row of their sequence in this step: the warp that read their window writes it back shifted.
+struct ConvPrepArgs {
+    int n, total_heads, base, C, K, n_inplace;
+    atx_conv_head_seg seg[ATX_HEAD_SEGS_MAX];
+    const float* src;
+    long long ld;
+    float* conv_state;
+    const int *positions, *slots, *tok_seq, *seq_start, *seq_pos0, *seq_slot;
+    int T, bs, rows_per;
+    float eps;
+};
+constexpr int kHeadTaps = 8;
+
+// One warp takes one head and rows_per consecutive rows, the taps' window in registers. A lane owns E elements in groups of VE
+// neighbours (VE = min(E, 4)), so a rotated pair lies inside a lane. KT: taps when it is a common number, 0: up to kHeadTaps.
+template <typename XT, int E, int KT>
+__global__ void __launch_bounds__(256)
+conv_head_prepare_kernel(const __grid_constant__ ConvPrepArgs a) {
+    constexpr int VE = E < 4 ? E : 4, NG = E / VE;
+    constexpr int MT = KT ? KT : kHeadTaps;
+    constexpr int NW = MT > 1 ? MT - 1 : 1;
+    const int K = KT ? KT : a.K;
+    pdl_launch_dependents();
+    const int lane = threadIdx.x & 31;
+    const long long wid = static_cast<long long>(blockIdx.x) * (blockDim.x >> 5) + (threadIdx.x >> 5);
+    const long long tile = wid / a.total_heads;
+    const int t0 = static_cast<int>(tile) * a.rows_per;
+    if (t0 >= a.T) return;
+    int hh = static_cast<int>(wid - tile * a.total_heads), si = 0;
+    while (si + 1 < a.n && hh >= a.seg[si].heads) {
+        hh -= a.seg[si].heads;
+        ++si;
+    }
+    const atx_conv_head_seg& s = a.seg[si];
+    const int width = s.width, half = s.rot_dims / 2;
+    const long long col = s.src_off + static_cast<long long>(hh) * width;   // source column of the head's first element
+    const long long ch = col - a.base;                                     // its channel in the state
+    const XT* w = reinterpret_cast<const XT*>(s.w) + static_cast<long long>(hh) * width * K;
+    bool on[NG];
+    int el[NG];   // first element of each of the lane's groups
+    float wt[MT][E];
+#pragma unroll
+    for (int g = 0; g < NG; ++g) {
+        el[g] = g * 32 * VE + lane * VE;
+        on[g] = el[g] < width;
+#pragma unroll
+        for (int e = 0; e < VE; ++e)
+#pragma unroll
+            for (int j = 0; j < MT; ++j)
+                wt[j][g * VE + e] = (on[g] && j < K) ? hld(w, static_cast<long long>(el[g] + e) * K + j) : 0.f;
+    }
+    pdl_wait();   // the taps are weights: fetched ahead of the wait for the projection
+    auto load = [&](const float* p, float (&v)[E]) {   // p: the head's first element of some row
+#pragma unroll
+        for (int g = 0; g < NG; ++g) {
+            if constexpr (VE == 4) {
+                const float4 f = on[g] ? *reinterpret_cast<const float4*>(p + el[g]) : make_float4(0.f, 0.f, 0.f, 0.f);
+                v[g * VE] = f.x, v[g * VE + 1] = f.y, v[g * VE + 2] = f.z, v[g * VE + 3] = f.w;
+            } else {
+                const float2 f = on[g] ? *reinterpret_cast<const float2*>(p + el[g]) : make_float2(0.f, 0.f);
+                v[g * VE] = f.x, v[g * VE + 1] = f.y;
+            }
+        }
+    };
+    auto put = [&](XT* p, const float (&v)[E]) {
+#pragma unroll
+        for (int g = 0; g < NG; ++g) {
+            if (!on[g]) continue;
+            if constexpr (VE == 4) {
+                hst4(p + el[g], 0, make_float4(v[g * VE], v[g * VE + 1], v[g * VE + 2], v[g * VE + 3]));
+            } else if constexpr (sizeof(XT) == 2) {
+                *reinterpret_cast<uint32_t*>(p + el[g]) = pack_bf16(v[g * VE], v[g * VE + 1]);
+            } else {
+                *reinterpret_cast<float2*>(p + el[g]) = make_float2(v[g * VE], v[g * VE + 1]);
+            }
+        }
+    };
+    float win[NW][E], cur[E], nxt[E];
+    load(a.src + static_cast<long long>(t0) * a.ld + col, nxt);
+    int prev_s = -1, prev_i = -2;
+    for (int r = 0; r < a.rows_per && t0 + r < a.T; ++r) {
+        const long long t = t0 + r;
+#pragma unroll
+        for (int e = 0; e < E; ++e) cur[e] = nxt[e];
+        if (r + 1 < a.rows_per && t + 1 < a.T) load(a.src + (t + 1) * a.ld + col, nxt);   // the next row while this one is worked on
+        const int sq = a.tok_seq[t], slot = a.slots[t];
+        if (sq < 0 || slot < 0) continue;   // padded row
+        const int i = static_cast<int>(t) - a.seq_start[sq];
+        float* st = a.conv_state + static_cast<long long>(a.seq_slot[sq]) * (K - 1) * a.C + ch;
+        if (sq != prev_s || i != prev_i + 1) {
+            const int pos0 = a.seq_pos0[sq];
+#pragma unroll
+            for (int j = 0; j < NW; ++j) {
+#pragma unroll
+                for (int e = 0; e < E; ++e) win[j][e] = 0.f;
+                if (j < K - 1) {
+                    const int rel = i - (K - 1) + j;   // row of the portion that tap j reads (negative: before it)
+                    if (rel >= 0)
+                        load(a.src + (t - i + rel) * a.ld + col, win[j]);
+                    else if (pos0 + rel >= 0)
+                        load(st + static_cast<long long>(K - 1 + rel) * a.C, win[j]);
+                }
+            }
+        }
+        float u[E];
+#pragma unroll
+        for (int e = 0; e < E; ++e) u[e] = 0.f;
+#pragma unroll
+        for (int j = 0; j < MT; ++j) {
+            if (j < K - 1) {
+#pragma unroll
+                for (int e = 0; e < E; ++e) u[e] = fmaf(wt[j][e], win[j < NW ? j : 0][e], u[e]);
+            } else if (j == K - 1) {
+#pragma unroll
+                for (int e = 0; e < E; ++e) u[e] = fmaf(wt[j][e], cur[e], u[e]);
+            }
+        }
+        // slide: entries 0 .. K - 2 hold the K - 1 inputs before the next row
+#pragma unroll
+        for (int j = 0; j + 1 < NW; ++j)
+            if (j < K - 2)
+#pragma unroll
+                for (int e = 0; e < E; ++e) win[j][e] = win[j + 1][e];
+#pragma unroll
+        for (int j = 0; j < NW; ++j)
+            if (j == K - 2)
+#pragma unroll
+                for (int e = 0; e < E; ++e) win[j][e] = cur[e];
+        prev_s = sq;
+        prev_i = i;
+        if (sq < a.n_inplace) {
+#pragma unroll
+            for (int j = 0; j < NW; ++j) {
+                if (j >= K - 1) continue;
+                float* p = st + static_cast<long long>(j) * a.C;
+#pragma unroll
+                for (int g = 0; g < NG; ++g) {
+                    if (!on[g]) continue;
+                    if constexpr (VE == 4)
+                        *reinterpret_cast<float4*>(p + el[g]) = make_float4(win[j][g * VE], win[j][g * VE + 1], win[j][g * VE + 2], win[j][g * VE + 3]);
+                    else
+                        *reinterpret_cast<float2*>(p + el[g]) = make_float2(win[j][g * VE], win[j][g * VE + 1]);
+                }
+            }
+        }
+        const int blk = slot / a.bs, off = slot - blk * a.bs;
+        const long long page = ((static_cast<long long>(blk) * s.heads + hh) * a.bs + off) * width;
+        if (s.raw_dst) put(reinterpret_cast<XT*>(s.raw_dst) + page, u);
+        if (half > 0) {
+            const float* cs = s.rot + static_cast<long long>(a.positions[t]) * s.rot_dims;
+#pragma unroll
+            for (int g = 0; g < NG; ++g)
+#pragma unroll
+                for (int e = 0; e < VE; e += 2) {
+                    const int p = (el[g] + e) >> 1;
+                    if (p < half) {
+                        const float c = cs[p], sn = cs[half + p], x = u[g * VE + e], y = u[g * VE + e + 1];
+                        u[g * VE + e] = fmaf(x, c, -(y * sn));
+                        u[g * VE + e + 1] = fmaf(y, c, x * sn);
+                    }
+                }
+        }
+        if (s.norm) {
+            float ss = 0.f;
+#pragma unroll
+            for (int e = 0; e < E; ++e) ss = fmaf(u[e], u[e], ss);   // elements past the head are zero
+            const float rs = rsqrtf(warp_sum(ss) / static_cast<float>(width) + a.eps);
+#pragma unroll
+            for (int e = 0; e < E; ++e) u[e] *= rs;
+        }
+        put(reinterpret_cast<XT*>(s.dst) + (s.dst_kind == ATX_HEAD_DST_PAGES ? page : t * s.dst_ld + static_cast<long long>(hh) * width), u);
+    }
+}
+
+// Any width, alignment and number of taps: a warp per (row, head), the convolved head staged in shared memory.
+template <typename XT>
+__global__ void __launch_bounds__(256)
+conv_head_prepare_any_kernel(const __grid_constant__ ConvPrepArgs a, int stage) {
+    extern __shared__ float sconv[];   // [warps][stage]
+    pdl_launch_dependents();
+    pdl_wait();
+    const int lane = threadIdx.x & 31;
+    float* u = sconv + (threadIdx.x >> 5) * stage;
+    const long long wid = static_cast<long long>(blockIdx.x) * (blockDim.x >> 5) + (threadIdx.x >> 5);
+    const long long t = wid / a.total_heads;
+    if (t >= a.T) return;
+    int hh = static_cast<int>(wid - t * a.total_heads), si = 0;
+    while (si + 1 < a.n && hh >= a.seg[si].heads) {
+        hh -= a.seg[si].heads;
+        ++si;
+    }
+    const atx_conv_head_seg& s = a.seg[si];
+    const int sq = a.tok_seq[t], slot = a.slots[t], K = a.K;
+    if (sq < 0 || slot < 0) return;
+    const int width = s.width, half = s.rot_dims / 2;
+    const long long col = s.src_off + static_cast<long long>(hh) * width, ch = col - a.base;
+    const XT* w = reinterpret_cast<const XT*>(s.w) + static_cast<long long>(hh) * width * K;
+    const int i = static_cast<int>(t) - a.seq_start[sq], pos0 = a.seq_pos0[sq];
+    float* st = a.conv_state + static_cast<long long>(a.seq_slot[sq]) * (K - 1) * a.C + ch;
+    const bool inplace = sq < a.n_inplace;
+    const int blk = slot / a.bs, off = slot - blk * a.bs;
+    const long long page = ((static_cast<long long>(blk) * s.heads + hh) * a.bs + off) * width;
+    for (int c = lane; c < width; c += 32) {
+        float acc = 0.f;
+        for (int j = 0; j < K; ++j) {
+            const int rel = i - (K - 1 - j);
+            float v = 0.f;
+            if (rel >= 0)
+                v = a.src[(t - i + rel) * a.ld + col + c];
+            else if (pos0 + rel >= 0)
+                v = st[static_cast<long long>(K - 1 + rel) * a.C + c];
+            if (inplace && j > 0) st[static_cast<long long>(j - 1) * a.C + c] = v;   // entry j - 1 has been read already
+            acc = fmaf(hld(w, static_cast<long long>(c) * K + j), v, acc);
+        }
+        u[c] = acc;
+        if (s.raw_dst) hst(reinterpret_cast<XT*>(s.raw_dst) + page, c, acc);
+    }
+    __syncwarp();
+    const float* cs = half > 0 ? s.rot + static_cast<long long>(a.positions[t]) * s.rot_dims : nullptr;
+    for (int p = lane; p < half; p += 32) {
+        const float c = cs[p], sn = cs[half + p], x = u[2 * p], y = u[2 * p + 1];
+        u[2 * p] = fmaf(x, c, -(y * sn));
+        u[2 * p + 1] = fmaf(y, c, x * sn);
+    }
+    __syncwarp();
+    float rs = 1.f;
+    if (s.norm) {
+        float ss = 0.f;
+        for (int c = lane; c < width; c += 32) ss = fmaf(u[c], u[c], ss);
+        rs = rsqrtf(warp_sum(ss) / static_cast<float>(width) + a.eps);
+    }
+    XT* dst = reinterpret_cast<XT*>(s.dst) + (s.dst_kind == ATX_HEAD_DST_PAGES ? page : t * s.dst_ld + static_cast<long long>(hh) * width);
+    for (int c = lane; c < width; c += 32) hst(dst, c, u[c] * rs);
+}
+
+// ---- cap on logits ---------------------------------------------------------------------------------------------------------------
+__global__ void __launch_bounds__(256)
+soft_cap_kernel(float* __restrict__ x, long long ld, int T, int N, float cap) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const long long n = static_cast<long long>(T) * N;
+    for (long long e = static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x; e < n;
+         e += static_cast<long long>(gridDim.x) * blockDim.x) {
+        const long long t = e / N;
+        float* p = x + t * ld + (e - t * N);
+        *p = cap * tanhf(*p / cap);
+    }
+}
+
 // ---- per-head matrix product --------------------------------------------------------------------------------------------
 // out[t, h * os + n] = (sum_k X[t, x_off + h * xs + k] W[(h N + n) ldw + k]) (* sigmoid(gate[t, h N + n])).
 // FMA pipe, fp32 accumulation in a fixed order; 64 x 64 outputs per CTA, 4 x 4 per thread; blockIdx.z = head.
@@ -514,6 +772,98 @@ int atx_head_prepare(const float* src, long long ld, const atx_head_seg* segs, i
     else
         ATX_HEADOPS_XT(dtype, ATX_CUDA(cudaLaunchKernelEx(&cfg, head_prepare_kernel<XT, false>, src, ld, positions, slots, T,
                                                           block_size, eps, a)));
+    return ATX_OK;
+}
+
+int atx_conv_head_prepare(const float* src, long long ld, const atx_conv_head_seg* segs, int n_segs, int K, float* conv_state,
+                          int C, int n_inplace, const int* positions, const int* slots, const int* tok_seq,
+                          const int* seq_start, const int* seq_pos0, const int* seq_slot, int T, int block_size, float eps,
+                          int dtype, int flags, atx_stream_t stream) {
+    ATX_REQUIRE(src && segs && positions && slots && tok_seq && seq_start && seq_pos0 && seq_slot && (K == 1 || conv_state),
+                "atx_conv_head_prepare: null pointer");
+    ATX_REQUIRE(T > 0 && n_segs > 0 && n_segs <= ATX_HEAD_SEGS_MAX && K >= 1 && block_size > 0 && n_inplace >= 0,
+                "atx_conv_head_prepare: T=%d, %d segments (1..%d), %d taps", T, n_segs, ATX_HEAD_SEGS_MAX, K);
+    ConvPrepArgs a = {};
+    a.n = n_segs, a.base = segs[0].src_off, a.C = C, a.K = K, a.n_inplace = n_inplace;
+    a.src = src, a.ld = ld, a.conv_state = conv_state;
+    a.positions = positions, a.slots = slots, a.tok_seq = tok_seq, a.seq_start = seq_start, a.seq_pos0 = seq_pos0, a.seq_slot = seq_slot;
+    a.T = T, a.bs = block_size, a.eps = eps;
+    auto al16 = [](const void* p) { return reinterpret_cast<uintptr_t>(p) % 16 == 0; };
+    int widest = 0, all = 0;   // all: OR of every width, offset and pitch
+    bool aligned = al16(src) && al16(conv_state) && ld % 4 == 0 && C % 4 == 0;
+    for (int i = 0; i < n_segs; ++i) {
+        const atx_conv_head_seg& s = segs[i];
+        ATX_REQUIRE(s.heads > 0 && s.width > 0 && s.w && s.dst && s.src_off >= a.base &&
+                        s.src_off - a.base + static_cast<long long>(s.heads) * s.width <= C,
+                    "atx_conv_head_prepare: segment %d: heads=%d width=%d outside the %d channels", i, s.heads, s.width, C);
+        ATX_REQUIRE(s.rot_dims >= 0 && s.rot_dims % 2 == 0 && s.rot_dims <= s.width && (s.rot_dims == 0 || s.rot),
+                    "atx_conv_head_prepare: segment %d: rotation of %d of %d elements needs an even count and a table", i, s.rot_dims,
+                    s.width);
+        ATX_REQUIRE(s.dst_kind == ATX_HEAD_DST_PAGES || (s.dst_kind == ATX_HEAD_DST_ROWS && s.dst_ld >= static_cast<long long>(s.heads) * s.width),
+                    "atx_conv_head_prepare: segment %d: bad destination", i);
+        a.seg[i] = s;
+        a.total_heads += s.heads;
+        widest = s.width > widest ? s.width : widest;
+        all |= s.width | s.src_off | (s.dst_kind == ATX_HEAD_DST_ROWS ? static_cast<int>(s.dst_ld & 7) : 0);
+        aligned = aligned && al16(s.dst) && al16(s.raw_dst);
+    }
+    const bool fast = aligned && (all & 3) == 0 && widest <= 256 && K <= kHeadTaps;
+    cudaLaunchConfig_t cfg = {};
+    cudaLaunchAttribute attr[1];
+    cfg.stream = reinterpret_cast<cudaStream_t>(stream);
+    set_pdl_attr(cfg, attr, flags);
+    if (fast) {
+        a.rows_per = T >= 256 ? 16 : 1;
+        const long long warps = static_cast<long long>((T + a.rows_per - 1) / a.rows_per) * a.total_heads;
+        const int per = T >= 256 ? 8 : 4;   // decode-sized: smaller CTAs spread over more SMs
+        cfg.gridDim = dim3(static_cast<unsigned>((warps + per - 1) / per));
+        cfg.blockDim = dim3(32 * per);
+#define ATX_CONV_HEADS(E_, KT_) ATX_HEADOPS_XT(dtype, ATX_CUDA(cudaLaunchKernelEx(&cfg, conv_head_prepare_kernel<XT, E_, KT_>, a)))
+#define ATX_CONV_HEADS_E(E_)              \
+    do {                                  \
+        if (K == 4)                       \
+            ATX_CONV_HEADS(E_, 4);        \
+        else if (K == 3)                  \
+            ATX_CONV_HEADS(E_, 3);        \
+        else if (K == 2)                  \
+            ATX_CONV_HEADS(E_, 2);        \
+        else                              \
+            ATX_CONV_HEADS(E_, 0);        \
+    } while (0)
+        if (widest <= 64)
+            ATX_CONV_HEADS_E(2);
+        else if (widest <= 128)
+            ATX_CONV_HEADS_E(4);
+        else
+            ATX_CONV_HEADS_E(8);
+#undef ATX_CONV_HEADS_E
+#undef ATX_CONV_HEADS
+        return ATX_OK;
+    }
+    ATX_REQUIRE(widest <= 12000, "atx_conv_head_prepare: heads of %d elements (at most 12000)", widest);
+    a.rows_per = 1;
+    int per = 12000 / widest;
+    per = per > 8 ? 8 : (per < 1 ? 1 : per);
+    const long long warps = static_cast<long long>(T) * a.total_heads;
+    cfg.gridDim = dim3(static_cast<unsigned>((warps + per - 1) / per));
+    cfg.blockDim = dim3(32 * per);
+    cfg.dynamicSmemBytes = sizeof(float) * static_cast<size_t>(per) * widest;
+    ATX_HEADOPS_XT(dtype, ATX_CUDA(cudaLaunchKernelEx(&cfg, conv_head_prepare_any_kernel<XT>, a, widest)));
+    return ATX_OK;
+}
+
+int atx_soft_cap(float* x, long long ld, int T, int N, float cap, int flags, atx_stream_t stream) {
+    ATX_REQUIRE(x && T > 0 && N > 0 && ld >= N && cap > 0.f, "atx_soft_cap: bad arguments T=%d N=%d ld=%lld cap=%g", T, N, ld, cap);
+    const long long n = static_cast<long long>(T) * N;
+    long long blocks = (n + 256 * 4 - 1) / (256 * 4);
+    if (blocks > 148 * 16) blocks = 148 * 16;
+    cudaLaunchConfig_t cfg = {};
+    cudaLaunchAttribute attr[1];
+    cfg.gridDim = dim3(static_cast<unsigned>(blocks));
+    cfg.blockDim = dim3(256);
+    cfg.stream = reinterpret_cast<cudaStream_t>(stream);
+    set_pdl_attr(cfg, attr, flags);
+    ATX_CUDA(cudaLaunchKernelEx(&cfg, soft_cap_kernel, x, ld, T, N, cap));
     return ATX_OK;
 }
 

@@ -1,7 +1,7 @@
 // Mixture of experts: routing, the plan that sorts (token, choice) pairs by expert, the experts' matrix products over
 // their own rows, and the weighted sum.
-//   route    soft-max over the router's outputs in fp32; the `top` largest of score + correction are chosen (lowest
-//            index on ties), their weight is the plain score times a constant. One warp per token.
+//   route    soft-max over the router's outputs, or a sigmoid of each, in fp32; the `top` largest of score + correction are
+//            chosen (lowest index on ties), their weight is the plain score times a constant. One warp per token.
 //   plan     one CTA: rows per expert, their running offsets, a slot in the sorted order for every pair whose choice is a
 //            real expert (choices >= E stand for experts that return their input and take no slot), and the list of
 //            (expert, first slot) tiles the products run over. Which slot a pair gets inside its expert's range depends on
@@ -9,7 +9,8 @@
 //   product  out[slot, :] = A[row(slot), :] W_e^T for the slots of expert e, a tile of 64 slots x 64 outputs per CTA; CTAs
 //            past the plan's tile count leave at once, so the launch needs no count on the host. bf16 on the tensor cores
 //            (mma.sync m16n8k16, fp32 accumulation), fp32 on the FMA pipe. With `gated`, W_e holds N gate rows then N up
-//            rows and the CTA forms silu(gate) * up before it stores.
+//            rows and the CTA forms silu(gate) * up before it stores; an expert without a gate may have its activation
+//            max(z, 0)^2 applied before the store.
 //   combine  y[t] = shared_gate * y[t] + sum_k w[t, k] * (choice >= E ? x[t] : product[slot(t, k)]).
 #include "common.cuh"
 
@@ -43,7 +44,7 @@ constexpr int kRouteMax = 16;   // router outputs per lane: up to 512 outputs
 
 __global__ void __launch_bounds__(128)
 moe_route_kernel(const float* __restrict__ logits, long long ld, const float* __restrict__ correction, int R, int top,
-                 float scale, int* __restrict__ sel, float* __restrict__ wgt, int T, int normalize) {
+                 float scale, int* __restrict__ sel, float* __restrict__ wgt, int T, int normalize, int score, int power) {
     pdl_launch_dependents();
     pdl_wait();
     const int lane = threadIdx.x & 31;
@@ -58,21 +59,32 @@ moe_route_kernel(const float* __restrict__ logits, long long ld, const float* __
         s[i] = e < R ? z[e] : -INFINITY;
         mx = fmaxf(mx, s[i]);
     }
-    mx = warp_max(mx);
-    float sum = 0.f;
+    if (score == ATX_MOE_SIGMOID) {
+        // Without a correction the logits order the experts: a sigmoid that has reached 1 in fp32 no longer tells them apart.
 #pragma unroll
-    for (int i = 0; i < kRouteMax; ++i) {
-        const int e = lane + 32 * i;
-        s[i] = e < R ? expf(s[i] - mx) : 0.f;
-        sum += s[i];
-    }
-    sum = warp_sum(sum);
-    const float inv = 1.f / sum;
+        for (int i = 0; i < kRouteMax; ++i) {
+            const int e = lane + 32 * i;
+            const float zi = s[i];
+            s[i] = e < R ? 1.f / (1.f + expf(-zi)) : 0.f;
+            c[i] = e < R ? (correction ? s[i] + correction[e] : zi) : -INFINITY;
+        }
+    } else {
+        mx = warp_max(mx);
+        float sum = 0.f;
 #pragma unroll
-    for (int i = 0; i < kRouteMax; ++i) {
-        const int e = lane + 32 * i;
-        s[i] *= inv;
-        c[i] = e < R ? s[i] + (correction ? correction[e] : 0.f) : -INFINITY;
+        for (int i = 0; i < kRouteMax; ++i) {
+            const int e = lane + 32 * i;
+            s[i] = e < R ? expf(s[i] - mx) : 0.f;
+            sum += s[i];
+        }
+        sum = warp_sum(sum);
+        const float inv = 1.f / sum;
+#pragma unroll
+        for (int i = 0; i < kRouteMax; ++i) {
+            const int e = lane + 32 * i;
+            s[i] *= inv;
+            c[i] = e < R ? s[i] + (correction ? correction[e] : 0.f) : -INFINITY;
+        }
     }
     float chosen = 0.f;   // sum of the chosen scores
     for (int k = 0; k < top; ++k) {
@@ -96,12 +108,16 @@ moe_route_kernel(const float* __restrict__ logits, long long ld, const float* __
         chosen += bs;
         if (lane == 0) {
             sel[t * top + k] = bi;
-            wgt[t * top + k] = normalize ? bs : bs * scale;
+            const float w = bs * scale;
+            wgt[t * top + k] = normalize ? bs : (power == 2 ? w * w : w);
         }
     }
     if (normalize && lane == 0) {   // weights = chosen scores divided by their sum, times scale
         const float inv_c = 1.f / (chosen + 1e-20f);
-        for (int k = 0; k < top; ++k) wgt[t * top + k] = wgt[t * top + k] * inv_c * scale;
+        for (int k = 0; k < top; ++k) {
+            const float w = wgt[t * top + k] * inv_c * scale;
+            wgt[t * top + k] = power == 2 ? w * w : w;
+        }
     }
 }
 
@@ -173,7 +189,7 @@ __global__ void __launch_bounds__(128)
 moe_gemm_tc_kernel(const __nv_bfloat16* __restrict__ A, long long lda, const int* __restrict__ perm, int top, int gather,
                    const __nv_bfloat16* __restrict__ W, long long expert_stride, long long ldw, void* __restrict__ out,
                    long long ldo, int N, int K, const int* __restrict__ seg_off, const int* __restrict__ tiles,
-                   int interleaved) {
+                   int interleaved, int relu2) {
     constexpr int NW = GATED ? 2 : 1;
     constexpr int kStageElems = (BM + NW * kET) * kELD;
     extern __shared__ __align__(16) unsigned char moe_smem[];
@@ -276,6 +292,9 @@ moe_gemm_tc_kernel(const __nv_bfloat16* __restrict__ A, long long lda, const int
                 if (GATED) {
                     const float g = acc[0][nb][2 * rr + q], u = acc[NW - 1][nb][2 * rr + q];
                     reinterpret_cast<__nv_bfloat16*>(out)[p * ldo + n] = __float2bfloat16_rn(g / (1.f + expf(-g)) * u);
+                } else if (relu2) {
+                    const float z = fmaxf(acc[0][nb][2 * rr + q], 0.f);
+                    reinterpret_cast<__nv_bfloat16*>(out)[p * ldo + n] = __float2bfloat16_rn(z * z);
                 } else {
                     reinterpret_cast<float*>(out)[p * ldo + n] = acc[0][nb][2 * rr + q];
                 }
@@ -289,7 +308,7 @@ template <typename XT, bool GATED>
 __global__ void __launch_bounds__(256)
 moe_gemm_fma_kernel(const XT* __restrict__ A, long long lda, const int* __restrict__ perm, int top, int gather,
                     const XT* __restrict__ W, long long expert_stride, long long ldw, void* __restrict__ out, long long ldo,
-                    int N, int K, const int* __restrict__ seg_off, const int* __restrict__ tiles, int interleaved) {
+                    int N, int K, const int* __restrict__ seg_off, const int* __restrict__ tiles, int interleaved, int relu2) {
     constexpr int KC = 16;
     __shared__ float sa[KC][kET + 1];
     __shared__ float sw[GATED ? 2 : 1][KC][kET + 1];
@@ -355,6 +374,9 @@ moe_gemm_fma_kernel(const XT* __restrict__ A, long long lda, const int* __restri
             if (GATED) {
                 const float g = acc[0][i][j], u = acc[GATED ? 1 : 0][i][j];
                 mst(reinterpret_cast<XT*>(out), p * ldo + n, g / (1.f + expf(-g)) * u);
+            } else if (relu2) {
+                const float z = fmaxf(acc[0][i][j], 0.f);
+                mst(reinterpret_cast<XT*>(out), p * ldo + n, z * z);
             } else {
                 reinterpret_cast<float*>(out)[p * ldo + n] = acc[0][i][j];
             }
@@ -451,6 +473,13 @@ int atx_moe_route(const float* logits, long long ld, const float* correction, in
 
 int atx_moe_route_opts(const float* logits, long long ld, const float* correction, int R, int top, float scale,
                        int normalize, int* sel, float* wgt, int T, int flags, atx_stream_t stream) {
+    return atx_moe_route_scored(logits, ld, correction, R, top, scale, normalize, ATX_MOE_SOFTMAX, 1, sel, wgt, T, flags, stream);
+}
+
+int atx_moe_route_scored(const float* logits, long long ld, const float* correction, int R, int top, float scale,
+                         int normalize, int score, int power, int* sel, float* wgt, int T, int flags, atx_stream_t stream) {
+    ATX_REQUIRE((score == ATX_MOE_SOFTMAX || score == ATX_MOE_SIGMOID) && (power == 1 || power == 2),
+                "atx_moe_route: score=%d power=%d", score, power);
     ATX_REQUIRE(logits && sel && wgt, "atx_moe_route: null pointer");
     ATX_REQUIRE(T > 0 && R > 0 && R <= 32 * kRouteMax && top > 0 && top <= R && ld >= R,
                 "atx_moe_route: bad shape T=%d outputs=%d (<= %d) top=%d ld=%lld", T, R, 32 * kRouteMax, top, ld);
@@ -460,7 +489,8 @@ int atx_moe_route_opts(const float* logits, long long ld, const float* correctio
     cfg.blockDim = dim3(128);
     cfg.stream = reinterpret_cast<cudaStream_t>(stream);
     set_pdl_moe(cfg, attr, flags);
-    ATX_CUDA(cudaLaunchKernelEx(&cfg, moe_route_kernel, logits, ld, correction, R, top, scale, sel, wgt, T, normalize));
+    ATX_CUDA(cudaLaunchKernelEx(&cfg, moe_route_kernel, logits, ld, correction, R, top, scale, sel, wgt, T, normalize, score,
+                                power));
     return ATX_OK;
 }
 
@@ -489,6 +519,8 @@ int atx_moe_expert_gemm(const void* A, long long lda, const int* perm, int top, 
     ATX_REQUIRE(A && W && out && seg_off && tiles && (!gather || perm), "atx_moe_expert_gemm: null pointer");
     ATX_REQUIRE(N > 0 && K > 0 && max_tiles > 0 && max_tiles <= 65535 && top > 0 && ldw >= K && lda >= K && ldo >= N,
                 "atx_moe_expert_gemm: bad shape N=%d K=%d tiles=%d lda=%lld ldw=%lld ldo=%lld", N, K, max_tiles, lda, ldw, ldo);
+    const int relu2 = gated == ATX_MOE_ACT_RELU2 ? 1 : 0;   // no gate rows: the activation of an ungated expert
+    if (relu2) gated = 0;
     ATX_REQUIRE(!interleaved || (gated && N % 64 == 0), "atx_moe_expert_gemm: interleaved gate / up rows need N %% 64 == 0");
     ATX_REQUIRE(tile_rows == kET || (tile_rows == 16 && dtype == ATX_DT_BF16),
                 "atx_moe_expert_gemm: tiles of %d slots (64, or 16 for bf16)", tile_rows);
@@ -500,7 +532,7 @@ int atx_moe_expert_gemm(const void* A, long long lda, const int* perm, int top, 
 #define ATX_MOE_LAUNCH(KERNEL_, T_)                                                                                     \
     ATX_CUDA(cudaLaunchKernelEx(&cfg, KERNEL_, reinterpret_cast<const T_*>(A), lda, perm, top, gather,                \
                                 reinterpret_cast<const T_*>(W), expert_stride, ldw, out, ldo, N, K, seg_off, tiles,  \
-                                interleaved))
+                                interleaved, relu2))
     if (dtype == ATX_DT_BF16) {
         cfg.blockDim = dim3(128);
         const int smem = kEStages * ((tile_rows + (gated ? 2 : 1) * kET) * kELD) * 2;

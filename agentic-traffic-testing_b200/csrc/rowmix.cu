@@ -1,7 +1,9 @@
 // Row kernels in which a token reads its predecessor, and a feed-forward activation with row statistics:
 //   * embedding rows plus a row of a second table chosen by a hash of (previous token, token),
 //   * token shift: the normed row blended with the previous position's normed row, per channel,
-//   * a polynomial of unit-rms powers of the feed-forward's hidden row.
+//   * a polynomial of unit-rms powers of the feed-forward's hidden row,
+//   * the residual update of a parallel layer: stream + scale * (dense sublayer output + weighted expert outputs), embedding row
+//     and pass vector where a block of layers is entered, and the one or two norms of the next layer, in one pass over the row.
 // The predecessor of a step's first row comes from the sequence's state slot (the last token id; the last normed row of
 // every layer), which the CTA that read it then overwrites with the step's last row: reader and writer are the same
 // threads, so no second launch is needed. A sequence at position 0 has no predecessor whatever its slot holds.
@@ -197,6 +199,166 @@ poly_norm_act_kernel(const float* __restrict__ z, long long ldz, const float* __
     }
 }
 
+// ---- residual update of a parallel layer ------------------------------------------------------------------------------------
+// Per row t (r = rows ? rows[t] : t):
+//   v = h[r] (or the embedding row, table_mode 2) + y_scale * (y[r] + sum_k wgt[r, k] experts[slot_of[r, k]])
+//       + embedding row (table_mode 1) + vec;         h[r] = v (not with rows)
+//   out_x[t] = v / sqrt(mean(v^2) + eps) * (w_shift + w_x)     x = a, b
+// Both norms share the row's statistic. CTAs beyond T clear zero_ptr. NV > 0: NV vectors of four elements per thread, the row
+// stays in registers; NV = 0: any width and alignment, the row staged in shared memory.
+struct ParallelResidArgs {
+    float* h;
+    atx_resid_terms tm;
+    const void* w_a;
+    void* out_a;
+    const void* w_b;
+    void* out_b;
+    float w_shift, eps;
+    const int* rows;
+    int T, W;
+    uint4* zero_ptr;
+    long long zero_vecs;
+};
+constexpr int kResidTopMax = 64;
+
+__device__ __forceinline__ float row_sum(float v, float* red) {   // over the CTA; every thread gets the result
+    v = warp_sum(v);
+    if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = v;
+    __syncthreads();
+    float t = 0.f;
+    const int nw = (blockDim.x + 31) >> 5;
+    for (int i = 0; i < nw; ++i) t += red[i];
+    return t;
+}
+
+template <typename XT, int NV>
+__global__ void __launch_bounds__(1024)
+parallel_resid_norm_kernel(const __grid_constant__ ParallelResidArgs a) {
+    extern __shared__ __align__(16) float srow_p[];
+    __shared__ float red[32];
+    __shared__ float s_w[kResidTopMax];
+    __shared__ long long s_row[kResidTopMax];
+    pdl_launch_dependents();
+    const int W = a.W, W4 = W / 4;
+    const XT* wa = reinterpret_cast<const XT*>(a.w_a);
+    const XT* wb = reinterpret_cast<const XT*>(a.w_b);
+    const XT* vec = reinterpret_cast<const XT*>(a.tm.vec);
+    // one vector per thread (decode-sized steps): the weights, which no kernel writes, are fetched ahead of the wait
+    float4 wa4 = make_float4(0.f, 0.f, 0.f, 0.f), wb4 = wa4, vc4 = wa4;
+    if (NV == 1 && static_cast<int>(threadIdx.x) < W4 && static_cast<int>(blockIdx.x) < a.T) {
+        if (wa) wa4 = rld4(wa, threadIdx.x);
+        if (wb) wb4 = rld4(wb, threadIdx.x);
+        if (vec) vc4 = rld4(vec, threadIdx.x);
+    }
+    pdl_wait();
+    if (static_cast<int>(blockIdx.x) >= a.T) {
+        const long long nb = gridDim.x - a.T;
+        for (long long i = static_cast<long long>(blockIdx.x - a.T) * blockDim.x + threadIdx.x; i < a.zero_vecs;
+             i += nb * blockDim.x)
+            a.zero_ptr[i] = make_uint4(0, 0, 0, 0);
+        return;
+    }
+    const int t = blockIdx.x;
+    const long long r = a.rows ? a.rows[t] : t;
+    float* hr = a.h + r * W;
+    float* yr = a.tm.y ? a.tm.y + r * W : nullptr;
+    const int top = a.tm.experts ? a.tm.top : 0;
+    if (top) {
+        for (int k = threadIdx.x; k < top; k += blockDim.x) {
+            const int slot = a.tm.slot_of[r * top + k];
+            s_w[k] = slot >= 0 ? a.tm.wgt[r * top + k] : 0.f;
+            s_row[k] = slot >= 0 ? static_cast<long long>(slot) * a.tm.lde : -1;
+        }
+        __syncthreads();
+    }
+    const XT* er = nullptr;
+    if (a.tm.table_mode) {
+        int id = a.tm.ids[r];
+        id = id < 0 ? 0 : (id >= a.tm.vocab ? a.tm.vocab - 1 : id);
+        er = reinterpret_cast<const XT*>(a.tm.table) + static_cast<long long>(id) * W;
+    }
+    const bool start = a.tm.table_mode == 2, enter = a.tm.table_mode == 1;
+    const bool store = !a.rows && (yr || top || er || vec);
+    const float sc = a.tm.y_scale;
+    float ss = 0.f;
+    if constexpr (NV > 0) {
+        float4 v[NV];
+#pragma unroll
+        for (int n = 0; n < NV; ++n) {
+            const int i = threadIdx.x + n * blockDim.x;
+            v[n] = make_float4(0.f, 0.f, 0.f, 0.f);
+            if (i >= W4) continue;
+            v[n] = start ? rld4(er, i) : rld4(hr, i);
+            float4 add = make_float4(0.f, 0.f, 0.f, 0.f);
+            if (yr) {
+                add = rld4(yr, i);
+                if (a.tm.zero_y) rst4(yr, i, make_float4(0.f, 0.f, 0.f, 0.f));
+            }
+            for (int k = 0; k < top; ++k) {
+                if (s_row[k] < 0) continue;
+                const float4 e = *reinterpret_cast<const float4*>(a.tm.experts + s_row[k] + 4 * i);
+                const float w = s_w[k];
+                add.x = fmaf(w, e.x, add.x), add.y = fmaf(w, e.y, add.y), add.z = fmaf(w, e.z, add.z), add.w = fmaf(w, e.w, add.w);
+            }
+            v[n].x = fmaf(sc, add.x, v[n].x), v[n].y = fmaf(sc, add.y, v[n].y);
+            v[n].z = fmaf(sc, add.z, v[n].z), v[n].w = fmaf(sc, add.w, v[n].w);
+            if (enter) {
+                const float4 e = rld4(er, i);
+                v[n].x += e.x, v[n].y += e.y, v[n].z += e.z, v[n].w += e.w;
+            }
+            if (vec) {
+                const float4 c = NV == 1 ? vc4 : rld4(vec, i);
+                v[n].x += c.x, v[n].y += c.y, v[n].z += c.z, v[n].w += c.w;
+            }
+            if (store) rst4(hr, i, v[n]);
+            ss += v[n].x * v[n].x + v[n].y * v[n].y + v[n].z * v[n].z + v[n].w * v[n].w;
+        }
+        if (!a.out_a && !a.out_b) return;
+        const float rs = rsqrtf(row_sum(ss, red) / static_cast<float>(W) + a.eps), sh = a.w_shift;
+        XT* oa = reinterpret_cast<XT*>(a.out_a) + static_cast<long long>(t) * W;
+        XT* ob = reinterpret_cast<XT*>(a.out_b) + static_cast<long long>(t) * W;
+#pragma unroll
+        for (int n = 0; n < NV; ++n) {
+            const int i = threadIdx.x + n * blockDim.x;
+            if (i >= W4) continue;
+            const float4 u = make_float4(v[n].x * rs, v[n].y * rs, v[n].z * rs, v[n].w * rs);
+            if (a.out_a) {
+                const float4 g = NV == 1 ? wa4 : rld4(wa, i);
+                rst4(oa, i, make_float4(u.x * (sh + g.x), u.y * (sh + g.y), u.z * (sh + g.z), u.w * (sh + g.w)));
+            }
+            if (a.out_b) {
+                const float4 g = NV == 1 ? wb4 : rld4(wb, i);
+                rst4(ob, i, make_float4(u.x * (sh + g.x), u.y * (sh + g.y), u.z * (sh + g.z), u.w * (sh + g.w)));
+            }
+        }
+    } else {
+        for (int i = threadIdx.x; i < W; i += blockDim.x) {
+            float v = start ? rld(er, i) : hr[i], add = 0.f;
+            if (yr) {
+                add = yr[i];
+                if (a.tm.zero_y) yr[i] = 0.f;
+            }
+            for (int k = 0; k < top; ++k)
+                if (s_row[k] >= 0) add = fmaf(s_w[k], a.tm.experts[s_row[k] + i], add);
+            v = fmaf(sc, add, v);
+            if (enter) v += rld(er, i);
+            if (vec) v += rld(vec, i);
+            if (store) hr[i] = v;
+            srow_p[i] = v;
+            ss += v * v;
+        }
+        if (!a.out_a && !a.out_b) return;
+        const float rs = rsqrtf(row_sum(ss, red) / static_cast<float>(W) + a.eps);
+        XT* oa = reinterpret_cast<XT*>(a.out_a) + static_cast<long long>(t) * W;
+        XT* ob = reinterpret_cast<XT*>(a.out_b) + static_cast<long long>(t) * W;
+        for (int i = threadIdx.x; i < W; i += blockDim.x) {   // each thread re-reads what it wrote itself
+            const float u = srow_p[i] * rs;
+            if (a.out_a) rst(oa, i, u * (a.w_shift + rld(wa, i)));
+            if (a.out_b) rst(ob, i, u * (a.w_shift + rld(wb, i)));
+        }
+    }
+}
+
 }  // namespace atx
 
 using namespace atx;
@@ -254,6 +416,55 @@ int atx_poly_norm_act(const float* z, long long ldz, const float* coef, void* ou
     set_pdl_row(cfg, attr, flags);
     ATX_ROW_XT(dtype, ATX_CUDA(cudaLaunchKernelEx(&cfg, poly_norm_act_kernel<XT>, z, ldz, coef, reinterpret_cast<XT*>(out), ldo,
                                                   F, eps)));
+    return ATX_OK;
+}
+
+int atx_parallel_resid_norm(float* h, const atx_resid_terms* terms, const void* w_a, void* out_a, const void* w_b, void* out_b,
+                            float w_shift, const int* rows, int T, int W, float eps, void* zero_ptr, long long zero_bytes,
+                            int dtype, int flags, atx_stream_t stream) {
+    ATX_REQUIRE(h && terms, "atx_parallel_resid_norm: null pointer");
+    const atx_resid_terms& tm = *terms;
+    ATX_REQUIRE(T > 0 && W > 0 && W <= 12288, "atx_parallel_resid_norm: bad shape T=%d W=%d (W <= 12288)", T, W);
+    ATX_REQUIRE((w_a == nullptr) == (out_a == nullptr) && (w_b == nullptr) == (out_b == nullptr),
+                "atx_parallel_resid_norm: a norm weight and its output come together");
+    ATX_REQUIRE(!tm.experts || (tm.wgt && tm.slot_of && tm.top > 0 && tm.top <= kResidTopMax && tm.lde >= W),
+                "atx_parallel_resid_norm: experts need weights, slots and 1..%d choices (got %d)", kResidTopMax, tm.top);
+    ATX_REQUIRE(tm.table_mode >= 0 && tm.table_mode <= 2 && (tm.table_mode == 0 || (tm.ids && tm.table && tm.vocab > 0)),
+                "atx_parallel_resid_norm: table_mode=%d needs ids and a table", tm.table_mode);
+    ATX_REQUIRE(zero_bytes >= 0 && zero_bytes % 16 == 0 && (zero_bytes == 0 || zero_ptr) && !(tm.zero_y && rows),
+                "atx_parallel_resid_norm: zero_bytes=%lld must be a non-negative multiple of 16 with a buffer; zero_y not with rows",
+                zero_bytes);
+    ParallelResidArgs a = {h, tm, w_a, out_a, w_b, out_b, w_shift, eps, rows, T, W, reinterpret_cast<uint4*>(zero_ptr), zero_bytes / 16};
+    auto al16 = [](const void* p) { return reinterpret_cast<uintptr_t>(p) % 16 == 0; };
+    const bool v4 = W % 4 == 0 && al16(h) && al16(tm.y) && al16(tm.experts) && (!tm.experts || tm.lde % 4 == 0) && al16(tm.table) &&
+                    al16(tm.vec) && al16(w_a) && al16(out_a) && al16(w_b) && al16(out_b);
+    // few rows: as many threads per row as it has vectors; many rows: 256 threads and several vectors each
+    const int W4 = W / 4;
+    const int want = T <= 512 ? (W4 + 31) / 32 * 32 : 256;
+    int threads = want > 1024 ? 1024 : (want < 64 ? 64 : want);
+    while ((W4 + threads - 1) / threads > 8) threads *= 2;
+    const int nv = (W4 + threads - 1) / threads;
+    long long zb = (a.zero_vecs + 256 * 8 - 1) / (256 * 8);
+    if (zb > 2048) zb = 2048;
+    cudaLaunchConfig_t cfg = {};
+    cudaLaunchAttribute attr[1];
+    cfg.gridDim = dim3(static_cast<unsigned>(T + zb));
+    cfg.blockDim = dim3(v4 ? threads : 256);
+    cfg.dynamicSmemBytes = v4 ? 0 : static_cast<size_t>(W) * 4;
+    cfg.stream = reinterpret_cast<cudaStream_t>(stream);
+    set_pdl_row(cfg, attr, flags);
+#define ATX_PAR_RESID(NV_) ATX_ROW_XT(dtype, ATX_CUDA(cudaLaunchKernelEx(&cfg, parallel_resid_norm_kernel<XT, NV_>, a)))
+    if (!v4)
+        ATX_PAR_RESID(0);
+    else if (nv <= 1)
+        ATX_PAR_RESID(1);
+    else if (nv == 2)
+        ATX_PAR_RESID(2);
+    else if (nv <= 4)
+        ATX_PAR_RESID(4);
+    else
+        ATX_PAR_RESID(8);
+#undef ATX_PAR_RESID
     return ATX_OK;
 }
 

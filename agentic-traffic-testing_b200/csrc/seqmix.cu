@@ -393,18 +393,21 @@ gated_norm_warp_kernel(const float* __restrict__ y, long long ldy, const float* 
     }
 }
 
+constexpr int kConvRows = 16, kConvMaxTaps = 8;
+
 // ---- short causal convolution + silu, step size and decay of the selective scan -------------------------------------
 // Channel c of row t: out = silu(b[c] + sum_j w[c][j] * in[row(t) - (K-1-j)]), the last tap being the row itself. Inputs
 // before the step's first row come from the carried window conv_state[slot][K-1][C] (raw inputs of the last K-1
 // positions), inputs before position 0 are zero. Columns [C, C + H) of the same launch compute, per head,
-// dt = softplus(raw + dt_bias) and the decay exp(-exp(A_log) * dt).
+// dt = softplus(raw + dt_bias) and the decay exp(-exp(A_log) * dt). Sequences [0, n_inplace) bring one row each: the thread
+// that read their window of a channel writes it back shifted by one, so decoded tokens need no second launch for the state.
 template <typename XT>
 __global__ void __launch_bounds__(256)
 conv_dt_kernel(const float* __restrict__ in, long long ld, int x_off, int dt_off, const XT* __restrict__ w,
                const XT* __restrict__ b, const XT* __restrict__ dt_bias, const XT* __restrict__ a_log,
-               const float* __restrict__ conv_state, float* __restrict__ xbc, float* __restrict__ dt_out,
+               float* __restrict__ conv_state, float* __restrict__ xbc, float* __restrict__ dt_out,
                float* __restrict__ decay_out, const int* __restrict__ tok_seq, const int* __restrict__ seq_start,
-               const int* __restrict__ seq_pos0, const int* __restrict__ seq_slot, int C, int H, int K) {
+               const int* __restrict__ seq_pos0, const int* __restrict__ seq_slot, int C, int H, int K, int n_inplace) {
     pdl_launch_dependents();
     pdl_wait();
     const long long t = blockIdx.x;
@@ -412,18 +415,32 @@ conv_dt_kernel(const float* __restrict__ in, long long ld, int x_off, int dt_off
     if (s < 0) return;
     const int i = static_cast<int>(t) - seq_start[s];
     const int pos0 = seq_pos0[s];
-    const float* st = conv_state + static_cast<long long>(seq_slot[s]) * (K - 1) * C;
+    float* st = conv_state + static_cast<long long>(seq_slot[s]) * (K - 1) * C;
+    const bool inplace = s < n_inplace;
     for (int c = blockIdx.y * blockDim.x + threadIdx.x; c < C + H; c += gridDim.y * blockDim.x) {
         if (c < C) {
             float acc = ldf(b, c);
-            for (int j = 0; j < K; ++j) {
+            auto tap = [&](int j) -> float {
                 const int rel = i - (K - 1 - j);
-                float v = 0.f;
-                if (rel >= 0)
-                    v = in[(t - i + rel) * ld + x_off + c];
-                else if (pos0 + rel >= 0)
-                    v = st[static_cast<long long>(K - 1 + rel) * C + c];
-                acc = fmaf(ldf(w, static_cast<long long>(c) * K + j), v, acc);
+                if (rel >= 0) return in[(t - i + rel) * ld + x_off + c];
+                return pos0 + rel >= 0 ? st[static_cast<long long>(K - 1 + rel) * C + c] : 0.f;
+            };
+            if (K <= kConvMaxTaps) {   // every tap is in flight before the first one is used
+                float v[kConvMaxTaps];
+#pragma unroll
+                for (int j = 0; j < kConvMaxTaps; ++j) v[j] = j < K ? tap(j) : 0.f;
+#pragma unroll
+                for (int j = 0; j < kConvMaxTaps; ++j)
+                    if (j < K) acc = fmaf(ldf(w, static_cast<long long>(c) * K + j), v[j], acc);
+#pragma unroll
+                for (int j = 1; j < kConvMaxTaps; ++j)
+                    if (inplace && j < K) st[static_cast<long long>(j - 1) * C + c] = v[j];
+            } else {
+                for (int j = 0; j < K; ++j) {
+                    const float v = tap(j);
+                    if (inplace && j > 0) st[static_cast<long long>(j - 1) * C + c] = v;   // entry j - 1 has been read already
+                    acc = fmaf(ldf(w, static_cast<long long>(c) * K + j), v, acc);
+                }
             }
             xbc[t * C + c] = silu_f(acc);
         } else {
@@ -436,20 +453,19 @@ conv_dt_kernel(const float* __restrict__ in, long long ld, int x_off, int dt_off
     }
 }
 
-// The same for prompt-sized steps: a CTA takes kConvRows consecutive rows x 256 channels and every thread walks its channel
+// For prompt-sized steps: a CTA takes kConvRows consecutive rows x 256 channels and every thread walks its channel
 // down the rows with the taps' window in registers, so that each input and each weight is read once per tile instead
 // of once per row (one CTA per row re-reads the K-1 earlier rows and all weights from L2). The window is refilled from
 // the rows before the tile, or from the carried state, wherever a sequence starts or the rows are not consecutive.
-constexpr int kConvRows = 16, kConvMaxTaps = 8;
-
 // KT: the number of taps when it is one of the common ones (loops and window fold at compile time), 0: read K.
 template <typename XT, int KT>
 __global__ void __launch_bounds__(256)
 conv_dt_tile_kernel(const float* __restrict__ in, long long ld, int x_off, int dt_off, const XT* __restrict__ w,
                     const XT* __restrict__ b, const XT* __restrict__ dt_bias, const XT* __restrict__ a_log,
-                    const float* __restrict__ conv_state, float* __restrict__ xbc, float* __restrict__ dt_out,
+                    float* __restrict__ conv_state, float* __restrict__ xbc, float* __restrict__ dt_out,
                     float* __restrict__ decay_out, const int* __restrict__ tok_seq, const int* __restrict__ seq_start,
-                    const int* __restrict__ seq_pos0, const int* __restrict__ seq_slot, int T, int C, int H, int K_rt) {
+                    const int* __restrict__ seq_pos0, const int* __restrict__ seq_slot, int T, int C, int H, int K_rt,
+                    int n_inplace) {
     constexpr int MT = KT ? KT : kConvMaxTaps;   // registers for taps and window
     const int K = KT ? KT : K_rt;
     pdl_launch_dependents();
@@ -519,6 +535,12 @@ conv_dt_tile_kernel(const float* __restrict__ in, long long ld, int x_off, int d
 #pragma unroll
         for (int j = 0; j < MT - 1; ++j)
             if (j == K - 2) win[j] = raw[r];
+        if (s < n_inplace) {   // a single-row sequence: the slid window is its new state
+            float* st = conv_state + static_cast<long long>(seq_slot[s]) * (K - 1) * C;
+#pragma unroll
+            for (int j = 0; j < MT - 1; ++j)
+                if (j < K - 1) st[static_cast<long long>(j) * C + c] = win[j];
+        }
         prev_s = s;
         prev_i = i;
     }
@@ -1072,6 +1094,14 @@ int atx_conv_dt(const float* in, long long ld, int x_off, int dt_off, const void
                 const void* a_log, const float* conv_state, float* xbc, float* dt_out, float* decay_out,
                 const int* tok_seq, const int* seq_start, const int* seq_pos0, const int* seq_slot, int T, int C, int H,
                 int K, int dtype, int flags, atx_stream_t stream) {
+    return atx_conv_dt_inplace(in, ld, x_off, dt_off, w, b, dt_bias, a_log, const_cast<float*>(conv_state), xbc, dt_out, decay_out,
+                               tok_seq, seq_start, seq_pos0, seq_slot, 0, T, C, H, K, dtype, flags, stream);
+}
+
+int atx_conv_dt_inplace(const float* in, long long ld, int x_off, int dt_off, const void* w, const void* b,
+                        const void* dt_bias, const void* a_log, float* conv_state, float* xbc, float* dt_out,
+                        float* decay_out, const int* tok_seq, const int* seq_start, const int* seq_pos0, const int* seq_slot,
+                        int n_inplace, int T, int C, int H, int K, int dtype, int flags, atx_stream_t stream) {
     ATX_REQUIRE(in && w && b && dt_bias && a_log && conv_state && xbc && dt_out && decay_out && tok_seq && seq_start &&
                     seq_pos0 && seq_slot,
                 "atx_conv_dt: null pointer");
@@ -1090,7 +1120,7 @@ int atx_conv_dt(const float* in, long long ld, int x_off, int dt_off, const void
                                &cfg, conv_dt_tile_kernel<XT, KT_>, in, ld, x_off, dt_off, reinterpret_cast<const XT*>(w), \
                                reinterpret_cast<const XT*>(b), reinterpret_cast<const XT*>(dt_bias),                      \
                                reinterpret_cast<const XT*>(a_log), conv_state, xbc, dt_out, decay_out, tok_seq,           \
-                               seq_start, seq_pos0, seq_slot, T, C, H, K)))
+                               seq_start, seq_pos0, seq_slot, T, C, H, K, n_inplace)))
         if (K == 4)
             ATX_CONV_TILE(4);
         else if (K == 3)
@@ -1106,7 +1136,7 @@ int atx_conv_dt(const float* in, long long ld, int x_off, int dt_off, const void
                                &cfg, conv_dt_kernel<XT>, in, ld, x_off, dt_off, reinterpret_cast<const XT*>(w),
                                reinterpret_cast<const XT*>(b), reinterpret_cast<const XT*>(dt_bias),
                                reinterpret_cast<const XT*>(a_log), conv_state, xbc, dt_out, decay_out, tok_seq,
-                               seq_start, seq_pos0, seq_slot, C, H, K)));
+                               seq_start, seq_pos0, seq_slot, C, H, K, n_inplace)));
     return ATX_OK;
 }
 

@@ -66,6 +66,8 @@ typedef struct atx_gemm_plan atx_gemm_plan;
 /* ATX_GEMM_SWIGLU_BF16 with clamps (same row layout, same split-K): out = g sigmoid(alpha g) (u + shift) with g = min(acc_gate,
  * limit), u = clamp(acc_up, -limit, limit); the constants are the plan's (atx_gemm_plan_set_gate). */
 #define ATX_GEMM_GLU_CLAMP_BF16 5
+/* out fp32 = limit tanh(acc / limit), limit from atx_gemm_plan_set_gate: the cap on a model's logits. No split-K. */
+#define ATX_GEMM_SOFTCAP_F32 6
 int atx_gemm_plan_create(atx_gemm_plan** plan, const void* W, long long N, long long K, const void* X,
                          long long T_cap, long long ldx);
 void atx_gemm_plan_destroy(atx_gemm_plan* plan);
@@ -469,6 +471,7 @@ int atx_moe_route(const float* logits, long long ld, const float* correction, in
  * [2 + 2 * max_tiles] int32: the tile count, a spare word, then (expert, first slot) per tile of tile_rows slots
  * (atx_moe_tile_rows() for atx_moe_expert_gemm, atx_gemm_grouped_tile_rows() for atx_gemm_run_grouped);
  * max_tiles = ceil(n_pairs / tile_rows) + E always suffices. */
+#define ATX_MOE_ACT_RELU2 2
 int atx_moe_tile_rows(void);
 int atx_moe_plan(const int* sel, int n_pairs, int E, int tile_rows, int* seg_off, int* perm, int* slot_of, int* tiles,
                  int flags, atx_stream_t stream);
@@ -479,7 +482,8 @@ int atx_moe_gather_rows(const void* x, long long ldx, const int* perm, int top, 
 /* out[slot, n] = sum_k A[row(slot), k] * W[e * expert_stride + n * ldw + k] for the slots of every expert e; row(slot) =
  * perm[slot] / top with gather != 0, else slot. gated == 0: fp32 out. gated != 0: W holds N gate rows then N up rows per
  * expert (interleaved != 0: blocks of 64 gate rows and 64 up rows in turn, the layout ATX_GEMM_SWIGLU_BF16 reads) and
- * out (element type) = silu(gate) * up. bf16 on the tensor cores, fp32 on the FMA pipe. tile_rows: the slots per tile the
+ * out (element type) = silu(gate) * up. gated == ATX_MOE_ACT_RELU2: N plain rows per expert, out (element type) =
+ * max(z, 0)^2. bf16 on the tensor cores, fp32 on the FMA pipe. tile_rows: the slots per tile the
  * plan was made with, atx_moe_tile_rows(), or 16 (bf16 only: decode-sized steps, more CTAs per SM). The grid covers
  * max_tiles tiles; CTAs beyond the plan's count return. */
 int atx_moe_expert_gemm(const void* A, long long lda, const int* perm, int top, int gather, const void* W,
@@ -539,6 +543,69 @@ int atx_gated_linear_recurrence_chunked(const float* q, long long ldq, const flo
 /* atx_moe_route with normalize != 0: wgt = score / (sum of the chosen scores + 1e-20) * scale. */
 int atx_moe_route_opts(const float* logits, long long ld, const float* correction, int R, int top, float scale,
                        int normalize, int* sel, float* wgt, int T, int flags, atx_stream_t stream);
+
+/* ---- Further mechanisms: parallel layers with two norms of one row, re-entered blocks of layers, queries and keys behind a
+ * short convolution, sigmoid routing, capped logits. (Lifuzen is built from these; every constant is an argument.) */
+
+/* What a parallel layer adds to the stream (see atx_parallel_resid_norm). y (nullable): the dense sublayers' output [T, W];
+ * zero_y != 0 clears each row once read. experts (nullable): expert outputs by slot (row pitch lde), slot_of / wgt [T, top] as
+ * atx_moe_plan / atx_moe_route* write them (slot -1: no contribution). table_mode 1: the embedding row of ids[r] is added;
+ * 2: the stream starts as that row (h is not read). vec (nullable, element type [W]) is added last. */
+typedef struct atx_resid_terms {
+    float* y;
+    const float* experts;
+    const float* wgt;
+    const int* slot_of;
+    const int* ids;
+    const void* table;
+    const void* vec;
+    long long lde;
+    float y_scale;
+    int zero_y, top, vocab, table_mode;
+} atx_resid_terms;
+/* v = h[r] + y_scale (y[r] + sum_k wgt[r, k] experts[slot_of[r, k]]) (+ table[ids[r]]) (+ vec), r = rows ? rows[t] : t; h[r] = v
+ * (without rows); out_a[t] = rms(v) (w_shift + w_a), out_b[t] = rms(v) (w_shift + w_b) (each nullable; one row statistic for
+ * both; w_shift 1 for weights stored around zero). Spare CTAs clear zero_ptr / zero_bytes (a multiple of 16). W <= 12288. */
+int atx_parallel_resid_norm(float* h, const atx_resid_terms* terms, const void* w_a, void* out_a, const void* w_b, void* out_b,
+                            float w_shift, const int* rows, int T, int W, float eps, void* zero_ptr, long long zero_bytes,
+                            int dtype, int flags, atx_stream_t stream);
+/* One slice of a projection row whose channels pass a causal convolution over time before they are used as heads: `heads` heads
+ * of `width` elements from column src_off on, taps w [heads * width, K] (last tap = the row itself; no bias, no activation).
+ * Per head, in this order: convolution; raw_dst (nullable, pages [blocks, heads, block_size, width]) receives the result as it
+ * is; the first rot_dims elements are rotated in adjacent pairs by the angles of rot [max_pos, rot_dims] (cosines, then sines)
+ * at the row's position; with norm the head is divided by its root mean square; it goes to rows (dst [T, dst_ld], head h at
+ * column h * width) or to pages (dst as raw_dst). */
+typedef struct atx_conv_head_seg {
+    int src_off, heads, width;
+    int norm, rot_dims, dst_kind;
+    const void* w;
+    const float* rot;
+    void* dst;
+    void* raw_dst;
+    long long dst_ld;
+} atx_conv_head_seg;
+/* The slices' channels are columns [segs[0].src_off, + C) of src (fp32 [T, ld]); the K - 1 rows before a step come from
+ * conv_state [slots, K - 1, C] fp32, rows before position 0 are zero. Sequences [0, n_inplace) bring exactly one row each and
+ * have their state shifted here; for the others atx_conv_state_update(src, ld, segs[0].src_off, ...) follows. */
+int atx_conv_head_prepare(const float* src, long long ld, const atx_conv_head_seg* segs, int n_segs, int K, float* conv_state,
+                          int C, int n_inplace, const int* positions, const int* slots, const int* tok_seq,
+                          const int* seq_start, const int* seq_pos0, const int* seq_slot, int T, int block_size, float eps,
+                          int dtype, int flags, atx_stream_t stream);
+/* atx_conv_dt that shifts the carried inputs of sequences [0, n_inplace) (one row each) itself; for the others
+ * atx_conv_state_update follows. */
+int atx_conv_dt_inplace(const float* in, long long ld, int x_off, int dt_off, const void* w, const void* b,
+                        const void* dt_bias, const void* a_log, float* conv_state, float* xbc, float* dt_out,
+                        float* decay_out, const int* tok_seq, const int* seq_start, const int* seq_pos0, const int* seq_slot,
+                        int n_inplace, int T, int C, int H, int K, int dtype, int flags, atx_stream_t stream);
+/* atx_moe_route_opts with a choice of score: soft-max over the outputs, or a sigmoid of each (without a correction the logits
+ * themselves then order the experts); power 2: wgt is squared. An expert that reads its weighted input, f(w x), equals w^2 f(x)
+ * for w >= 0 when f is W_down max(W_up x, 0)^2, so the weight can stay out of the expert's products. */
+#define ATX_MOE_SOFTMAX 0
+#define ATX_MOE_SIGMOID 1
+int atx_moe_route_scored(const float* logits, long long ld, const float* correction, int R, int top, float scale,
+                         int normalize, int score, int power, int* sel, float* wgt, int T, int flags, atx_stream_t stream);
+/* x[t, n] = cap tanh(x[t, n] / cap) in place, n < N. */
+int atx_soft_cap(float* x, long long ld, int T, int N, float cap, int flags, atx_stream_t stream);
 
 #ifdef __cplusplus
 }
