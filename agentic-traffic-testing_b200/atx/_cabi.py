@@ -52,6 +52,7 @@ EXPORTS = [
     "atx_gated_linear_recurrence", "atx_moe_route_opts", "atx_gemm_plan_set_gate",
     "atx_gated_linear_recurrence_chunked", "atx_gated_linear_recurrence_chunked_supported",
     "atx_parallel_resid_norm", "atx_conv_head_prepare", "atx_conv_dt_inplace", "atx_moe_route_scored", "atx_soft_cap",
+    "atx_moe_route_plan", "atx_gemm_run_grouped_small",
 ]
 ATTN_SOFTMAX = 0
 ATTN_SIGMOID = 1
@@ -241,6 +242,8 @@ def load() -> C.CDLL:
     lib.atx_conv_dt_inplace.argtypes = [vp, i64, i32, i32, vp, vp, vp, vp, vp, vp, vp, vp, vp, vp, vp, vp, i32, i32, i32, i32, i32,
                                         i32, i32, vp]
     lib.atx_moe_route_scored.argtypes = [vp, i64, vp, i32, i32, f32, i32, i32, i32, vp, vp, i32, i32, vp]
+    lib.atx_moe_route_plan.argtypes = [vp, i64, vp, i32, i32, f32, i32, i32, i32, i32, i32, i32, vp, vp, vp, vp, vp, vp, i32, vp]
+    lib.atx_gemm_run_grouped_small.argtypes = [vp, vp, i64, i32, i32, vp, vp, i32, vp, i32, i32, i32, vp]
     lib.atx_soft_cap.argtypes = [vp, i64, i32, i32, f32, i32, vp]
     for name in EXPORTS:  # fail at load time, not at first use, if the build is stale
         getattr(lib, name)

@@ -122,9 +122,8 @@ class UngatedExperts:
         F = max([int(m["expert"]["ff"]) for m in specs], default=1)
         P = T * top if specs else 1
         self.P = P
-        self.sms = torch.cuda.get_device_properties(dev).multi_processor_count
         self.tile_rows, self.big_rows = int(lib.atx_moe_tile_rows()), int(lib.atx_gemm_grouped_tile_rows())
-        self.max_tiles = max((P + self.tile_rows - 1) // self.tile_rows, (min(P, 64 * top) + 15) // 16) + E
+        self.max_tiles = (P + self.tile_rows - 1) // self.tile_rows + E
         self.max_big_tiles = (P + self.big_rows - 1) // self.big_rows + E
         self.sel = torch.zeros(P, dtype=i32, device=dev)
         self.wgt = torch.zeros(P, dtype=torch.float32, device=dev)
@@ -139,11 +138,12 @@ class UngatedExperts:
         self.xperm = torch.zeros(P if self.grouped else 1, W, dtype=xt, device=dev)
 
     def plans(self, w_up: torch.Tensor, w_down: torch.Tensor) -> Optional[dict]:
-        """GEMM plans of one layer for prompt-sized steps (w_up [E, F, W], w_down [E, W, F]), or None where the sizes have none."""
+        """GEMM plans of one layer (w_up [E, F, W], w_down [E, W, F]; the up product over gathered rows, and over the step's tokens as
+        they are), or None where the sizes have none."""
         E, F, W = w_up.shape
         if not (_use_tc(w_up.dtype, W) and F % 64 == 0):
             return None
-        return {"up": _cabi.GemmPlan(w_up.view(E * F, W), self.xperm),
+        return {"up": _cabi.GemmPlan(w_up.view(E * F, W), self.xperm), "up_tokens": _cabi.GemmPlan(w_up.view(E * F, W), self.xn),
                 "down": _cabi.GemmPlan(w_down.view(E * W, F), self.act[:self.P * F].view(self.P, F))}
 
     def run(self, logits: int, ld: int, top: int, w_up: torch.Tensor, w_down: torch.Tensor, plans: Optional[dict], T: int,
@@ -154,22 +154,33 @@ class UngatedExperts:
         E, F = int(w_up.shape[0]), int(w_up.shape[1])
         sel, so, pm, sl = (t.data_ptr() for t in (self.sel, self.seg_off, self.perm, self.slot_of))
         pairs, act, out, x = T * top, self.act.data_ptr(), self.out.data_ptr(), self.xn.data_ptr()
-        ck(lib.atx_moe_route_scored(logits, ld, None, E, top, 1.0, 0, _cabi.MOE_SIGMOID, 2, sel, self.wgt.data_ptr(), T, fl, st))
-        if plans is not None and not small:
-            # prompt-sized: gather every expert's rows, then both products on the tcgen05 GEMM over the plan's tiles
-            big, tb = min(self.max_big_tiles, (pairs + self.big_rows - 1) // self.big_rows + E), self.tiles_big.data_ptr()
-            ck(lib.atx_moe_plan(sel, pairs, E, self.big_rows, so, pm, sl, tb, fl, st))
-            ck(lib.atx_moe_gather_rows(x, W, pm, top, so, E, self.xperm.data_ptr(), W, pairs, W, dt, fl, st))
-            ck(lib.atx_gemm_run_grouped(plans["up"]._h, act, F, F, _cabi.GEMM_RELU2_BF16, so, tb, big, fl, st))
-            ck(lib.atx_gemm_run_grouped(plans["down"]._h, out, W, W, _cabi.GEMM_STORE_F32, so, tb, big, fl, st))
-            return 5
-        # decode-sized bf16 steps (one or two rows per expert): tiles of 16 slots let more CTAs share an SM where two per SM
-        # would need a second wave
-        ctas = min(E, pairs) * ((F + 63) // 64)
-        tr = 16 if (small and dt == _cabi.DT_BF16 and ctas > 2 * self.sms) else self.tile_rows
-        tiles, tl = min(self.max_tiles, (pairs + tr - 1) // tr + E), self.tiles.data_ptr()
-        ck(lib.atx_moe_plan(sel, pairs, E, tr, so, pm, sl, tl, fl, st))
-        ck(lib.atx_moe_expert_gemm(x, W, pm, top, 1, w_up.data_ptr(), F * W, W, act, F, F, W, _cabi.MOE_ACT_RELU2, 0, tr, so, tl,
-                                   tiles, dt, fl, st))
-        ck(lib.atx_moe_expert_gemm(act, F, None, top, 0, w_down.data_ptr(), W * F, F, out, W, W, F, 0, 0, tr, so, tl, tiles, dt, fl, st))
-        return 4
+        route = (logits, ld, None, E, top, 1.0, 0, _cabi.MOE_SIGMOID, 2)
+        wgt = self.wgt.data_ptr()
+        if small:
+            # decode-sized: one tile per chosen expert. With plans both products stream the chosen matrices on the tcgen05 kernel, the
+            # first one over the step's tokens as they are; without, 64-slot tiles on the expert kernel.
+            tiles, tl = min(E, pairs), self.tiles.data_ptr()
+            ck(lib.atx_moe_route_plan(*route, T, E, self.tile_rows, sel, wgt, so, pm, sl, tl, fl, st))
+            n = 1
+            if plans is not None:
+                ck(lib.atx_gemm_run_grouped_small(plans["up_tokens"]._h, act, F, F, _cabi.GEMM_RELU2_BF16, so, tl, tiles, pm, top, T, fl, st))
+                ck(lib.atx_gemm_run_grouped_small(plans["down"]._h, out, W, W, _cabi.GEMM_STORE_F32, so, tl, tiles, None, top, T, fl, st))
+                return n + 2
+        else:
+            ck(lib.atx_moe_route_scored(*route, sel, wgt, T, fl, st))
+            n = 2
+            if plans is not None:
+                # prompt-sized: gather every expert's rows, then both products on the persistent tcgen05 GEMM over the plan's tiles
+                big, tb = min(self.max_big_tiles, (pairs + self.big_rows - 1) // self.big_rows + E), self.tiles_big.data_ptr()
+                ck(lib.atx_moe_plan(sel, pairs, E, self.big_rows, so, pm, sl, tb, fl, st))
+                ck(lib.atx_moe_gather_rows(x, W, pm, top, so, E, self.xperm.data_ptr(), W, pairs, W, dt, fl, st))
+                ck(lib.atx_gemm_run_grouped(plans["up"]._h, act, F, F, _cabi.GEMM_RELU2_BF16, so, tb, big, fl, st))
+                ck(lib.atx_gemm_run_grouped(plans["down"]._h, out, W, W, _cabi.GEMM_STORE_F32, so, tb, big, fl, st))
+                return n + 3
+            tiles, tl = min(self.max_tiles, (pairs + self.tile_rows - 1) // self.tile_rows + E), self.tiles.data_ptr()
+            ck(lib.atx_moe_plan(sel, pairs, E, self.tile_rows, so, pm, sl, tl, fl, st))
+        ck(lib.atx_moe_expert_gemm(x, W, pm, top, 1, w_up.data_ptr(), F * W, W, act, F, F, W, _cabi.MOE_ACT_RELU2, 0, self.tile_rows, so,
+                                   tl, tiles, dt, fl, st))
+        ck(lib.atx_moe_expert_gemm(act, F, None, top, 0, w_down.data_ptr(), W * F, F, out, W, W, F, 0, 0, self.tile_rows, so, tl, tiles,
+                                   dt, fl, st))
+        return n + 2

@@ -452,6 +452,7 @@ class Program:
             self.state.append(st)
             self.conv_state.append(torch.zeros(S, max(1, int(c["conv"]) - 1), conv_channels(spec), dtype=f32, device=dev))
         # second stream for the feed-forward of decode-sized steps (see forward)
+        self.overlap_ffn = True
         self.side = torch.cuda.Stream(device=dev)
         self.ev_fork, self.ev_join = torch.cuda.Event(), torch.cuda.Event()
         # scratch of the decode attention's key slices: [tokens, heads, slices, value width + 2] fp32
@@ -604,7 +605,7 @@ class Program:
             # plan and expert products run on a second stream beside the mixer's chain of short kernels; the streams join in
             # front of the next residual kernel. Inside a captured graph these are two branches of the layer.
             fs, side = st, None
-            if E and small:
+            if E and small and self.overlap_ffn:
                 side = self.side
                 self.ev_fork.record(main)
                 side.wait_event(self.ev_fork)

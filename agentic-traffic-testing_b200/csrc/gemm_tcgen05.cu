@@ -79,11 +79,22 @@ __device__ __forceinline__ float dsmem_ld(uint32_t remote_addr) {
     return v;
 }
 
+// Groups of rows that each have their own block of W rows (a mixture of experts) in decode-sized steps: blockIdx.y is an entry
+// of the plan's tile list (one tile per group, since a group has at most TN rows). Without perm the group's rows of X lie back
+// to back from the tile's first slot; with perm X holds the step's TOKENS, every group multiplies all of them (at most TN = 64,
+// the weights are what is streamed) and only the group's own tokens are stored, at their slots.
+struct GroupedRows {
+    const int* tiles;
+    const int* seg;
+    const int* perm;
+    int top;
+};
+
 template <int TN>
 __global__ void __launch_bounds__(kGemmThreads)
 gemm_wt_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ CUtensorMap tmX,
                void* __restrict__ out, long long ldo, int T, int N, int kb_total, int kb_per_split,
-               int mode_in, int w_evict_first, int stages, GateParams gate_params) {
+               int mode_in, int w_evict_first, int stages, GateParams gate_params, GroupedRows grp) {
     const int mode = mode_in & 0xff;
     const bool ordered = (mode_in & 0x100) != 0;   // ATX_FLAG_ORDERED: split-K summed in a fixed order (below)
     // `stages` (<= Cfg::kStages) is the ring depth actually used: CTAs with few k-blocks get a smaller
@@ -101,7 +112,26 @@ gemm_wt_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
     const int warp = threadIdx.x >> 5;
     const int lane = threadIdx.x & 31;
     const int n0 = blockIdx.x * kBM;
-    const int t0 = blockIdx.y * TN;
+    int t0 = blockIdx.y * TN, w_row = n0;
+    __shared__ int s_row[64];   // grouped over token rows: output row of a token of this group (-1: not in the group)
+    if (grp.tiles) {
+        pdl_launch_dependents();
+        pdl_wait();   // the tile list is the upstream kernel's work
+        if (static_cast<int>(blockIdx.y) >= grp.tiles[0]) return;
+        const int e = grp.tiles[2 + 2 * blockIdx.y];
+        const int first = grp.tiles[3 + 2 * blockIdx.y], last = grp.seg[e + 1];
+        w_row = e * N + n0;
+        if (grp.perm) {
+            if (threadIdx.x < 64) s_row[threadIdx.x] = -1;
+            __syncthreads();
+            for (int p = first + threadIdx.x; p < last; p += kGemmThreads) s_row[grp.perm[p] / grp.top] = p;
+            t0 = 0;    // (read after the barriers of the prologue below)
+        } else {
+            t0 = first;
+            T = last;
+        }
+    }
+    const bool by_token = grp.tiles && grp.perm;
     const int kb_begin = blockIdx.z * kb_per_split;
     const int kb_end = min(kb_total, kb_begin + kb_per_split);
     const int nkb = kb_end - kb_begin;
@@ -138,7 +168,7 @@ gemm_wt_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
                 for (int i = 0; i < pre; ++i) {
                     mbar_expect_tx(&full_bar[i], Cfg::kStageBytes);
                     tma_load_2d(smem + i * Cfg::kStageBytes, &tmW, &full_bar[i],
-                                (kb_begin + i) * kBK, n0, polW);
+                                (kb_begin + i) * kBK, w_row, polW);
                 }
                 pdl_wait();
                 for (int i = 0; i < pre; ++i) {
@@ -151,7 +181,7 @@ gemm_wt_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
                     mbar_wait(&empty_bar[stage], phase);
                     uint8_t* st = smem + stage * Cfg::kStageBytes;
                     mbar_expect_tx(&full_bar[stage], Cfg::kStageBytes);
-                    tma_load_2d(st, &tmW, &full_bar[stage], (kb_begin + i) * kBK, n0, polW);
+                    tma_load_2d(st, &tmW, &full_bar[stage], (kb_begin + i) * kBK, w_row, polW);
                     tma_load_2d(st + Cfg::kStageBytesW, &tmX, &full_bar[stage], (kb_begin + i) * kBK,
                                 t0, kEvictLast);
                     if (++stage == stages) {
@@ -302,7 +332,9 @@ gemm_wt_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
 #pragma unroll
                     for (int j = 0; j < 16; ++j) {
                         const int t = t0 + c + j;
-                        if (t < T) o[static_cast<long long>(t) * ldo + n] = stored_value(__uint_as_float(v[j]), mode, gate_params);
+                        if (t >= T) continue;
+                        const int row = by_token ? s_row[c + j] : t;
+                        if (row >= 0) o[static_cast<long long>(row) * ldo + n] = stored_value(__uint_as_float(v[j]), mode, gate_params);
                     }
                 } else if (mode == ATX_GEMM_ADD_F32) {
                     // parked in shared memory (token-major) and added below, four consecutive outputs at a time
@@ -320,7 +352,9 @@ gemm_wt_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
                             a = fmaxf(a, 0.f);
                             a *= a;
                         }
-                        if (t < T) o[static_cast<long long>(t) * ldo + n] = __float2bfloat16_rn(a);
+                        if (t >= T) continue;
+                        const int row = by_token ? s_row[c + j] : t;
+                        if (row >= 0) o[static_cast<long long>(row) * ldo + n] = __float2bfloat16_rn(a);
                     }
                 }
             }
@@ -682,7 +716,8 @@ using namespace atx;
 
 template <int TN>
 static int launch_gemm(const atx_gemm_plan* p, int ti, void* out, long long ldo, int T, int mode,
-                       int splits, int pdl, cudaStream_t stream) {
+                       int splits, int pdl, cudaStream_t stream, const GroupedRows& grp = GroupedRows{}, int n_group = 0,
+                       int max_tiles = 0) {
     using Cfg = GemmCfg<TN>;
     static bool attr_done[64] = {false};  // per instantiation and device; benign race (idempotent call)
     int dev = 0;
@@ -700,7 +735,7 @@ static int launch_gemm(const atx_gemm_plan* p, int ti, void* out, long long ldo,
     // (a whole fp32 tile when the split-K cluster parks partial sums there)
     const bool ordered = (mode & 0x100) != 0;
     if (is_glu(mode & 0xff) || (mode & 0xff) == ATX_GEMM_ADD_F32 ||
-        ((mode & 0xff) == ATX_GEMM_RELU2_BF16 && zs > 1)) {
+        (((mode & 0xff) == ATX_GEMM_RELU2_BF16 || ordered) && zs > 1)) {
         // epilogues that park the tile in the (idle) stage buffers: half a tile for SwiGLU, a whole fp32 tile for the
         // split-K cluster reduction and for the 16-byte adds
         const bool whole = zs > 1 || (mode & 0xff) == ATX_GEMM_ADD_F32;
@@ -709,8 +744,9 @@ static int launch_gemm(const atx_gemm_plan* p, int ti, void* out, long long ldo,
     }
     const int smem_bytes = stages * Cfg::kStageBytes + 1024 + 256;
     cudaLaunchConfig_t cfg = {};
-    cfg.gridDim = dim3(static_cast<unsigned>((p->N + kBM - 1) / kBM), static_cast<unsigned>((T + TN - 1) / TN),
-                       static_cast<unsigned>(zs));
+    const long long rows = grp.tiles ? n_group : p->N;
+    cfg.gridDim = dim3(static_cast<unsigned>((rows + kBM - 1) / kBM),
+                       static_cast<unsigned>(grp.tiles ? max_tiles : (T + TN - 1) / TN), static_cast<unsigned>(zs));
     cfg.blockDim = dim3(kGemmThreads);
     cfg.dynamicSmemBytes = smem_bytes;
     cfg.stream = stream;
@@ -731,7 +767,7 @@ static int launch_gemm(const atx_gemm_plan* p, int ti, void* out, long long ldo,
     cfg.attrs = attr;
     cfg.numAttrs = na;
     ATX_CUDA(cudaLaunchKernelEx(&cfg, gemm_wt_kernel<TN>, p->tmW, p->tmX[ti], out, ldo, T,
-                                static_cast<int>(p->N), kb_total, kb_per, mode, p->w_evict_first, stages, p->gate));
+                                static_cast<int>(rows), kb_total, kb_per, mode, p->w_evict_first, stages, p->gate, grp));
     return ATX_OK;
 }
 
@@ -908,6 +944,29 @@ int atx_gemm_run_grouped(const atx_gemm_plan* p, void* out, long long ldo, int n
                 n_group);
     return launch_gemm_grouped<256>(p, 4, out, ldo, n_group, mode, seg_off, tiles, max_row_tiles, (flags & ATX_FLAG_PDL) ? 1 : 0,
                                     reinterpret_cast<cudaStream_t>(stream_));
+}
+
+int atx_gemm_run_grouped_small(const atx_gemm_plan* p, void* out, long long ldo, int n_group, int mode, const int* seg_off,
+                               const int* tiles, int max_tiles, const int* perm, int top, int T, int flags,
+                               atx_stream_t stream_) {
+    cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_);
+    ATX_REQUIRE(p && out && seg_off && tiles, "atx_gemm_run_grouped_small: null pointer");
+    ATX_REQUIRE(T > 0 && T <= 64 && max_tiles > 0 && max_tiles <= 65535 && top > 0, "atx_gemm_run_grouped_small: T=%d (1..64) tiles=%d", T,
+                max_tiles);
+    ATX_REQUIRE(n_group > 0 && p->N % n_group == 0 && ldo >= n_group,
+                "atx_gemm_run_grouped_small: W has %lld rows, not a multiple of %d per group (ldo=%lld)", p->N, n_group, ldo);
+    ATX_REQUIRE(mode == ATX_GEMM_STORE_F32 || mode == ATX_GEMM_STORE_BF16 || mode == ATX_GEMM_RELU2_BF16,
+                "atx_gemm_run_grouped_small: mode %d (plain stores and the squared ReLU)", mode);
+    // K-splits of a tile are a cluster whose leader sums them in a fixed order: as many as still fit one wave of two CTAs per SM
+    const long long ctas = static_cast<long long>((n_group + kBM - 1) / kBM) * max_tiles;
+    const int kb = static_cast<int>(p->K / kBK);
+    int splits = 1;
+    while (splits < 8 && ctas * splits * 2 <= 2ll * num_sms() && kb % (splits * 2) == 0 && kb / (splits * 2) >= 4) splits *= 2;
+    const int pdl = (flags & ATX_FLAG_PDL) ? 1 : 0, kmode = mode | (splits > 1 ? 0x100 : 0);
+    const GroupedRows grp{tiles, seg_off, perm, top};
+    if (T <= 16) return launch_gemm<16>(p, 0, out, ldo, T, kmode, splits, pdl, stream, grp, n_group, max_tiles);
+    if (T <= 32) return launch_gemm<32>(p, 1, out, ldo, T, kmode, splits, pdl, stream, grp, n_group, max_tiles);
+    return launch_gemm<64>(p, 2, out, ldo, T, kmode, splits, pdl, stream, grp, n_group, max_tiles);
 }
 
 }  // extern "C"

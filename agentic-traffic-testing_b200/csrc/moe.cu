@@ -42,15 +42,21 @@ static void set_pdl_moe(cudaLaunchConfig_t& cfg, cudaLaunchAttribute* attr, int 
 
 constexpr int kRouteMax = 16;   // router outputs per lane: up to 512 outputs
 
-__global__ void __launch_bounds__(128)
-moe_route_kernel(const float* __restrict__ logits, long long ld, const float* __restrict__ correction, int R, int top,
-                 float scale, int* __restrict__ sel, float* __restrict__ wgt, int T, int normalize, int score, int power) {
-    pdl_launch_dependents();
-    pdl_wait();
-    const int lane = threadIdx.x & 31;
-    const long long t = static_cast<long long>(blockIdx.x) * 4 + (threadIdx.x >> 5);
-    if (t >= T) return;
-    const float* z = logits + t * ld;
+struct RouteArgs {
+    const float* logits;
+    long long ld;
+    const float* correction;
+    int R, top;
+    float scale;
+    int normalize, score, power;
+};
+
+// One warp routes token t.
+__device__ __forceinline__ void route_token(const RouteArgs& a, long long t, int* __restrict__ sel, float* __restrict__ wgt) {
+    const int lane = threadIdx.x & 31, R = a.R, top = a.top, normalize = a.normalize, score = a.score, power = a.power;
+    const float scale = a.scale;
+    const float* correction = a.correction;
+    const float* z = a.logits + t * a.ld;
     float s[kRouteMax], c[kRouteMax];
     float mx = -INFINITY;
 #pragma unroll
@@ -121,18 +127,22 @@ moe_route_kernel(const float* __restrict__ logits, long long ld, const float* __
     }
 }
 
+__global__ void __launch_bounds__(128)
+moe_route_kernel(const __grid_constant__ RouteArgs a, int* __restrict__ sel, float* __restrict__ wgt, int T) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const long long t = static_cast<long long>(blockIdx.x) * 4 + (threadIdx.x >> 5);
+    if (t < T) route_token(a, t, sel, wgt);
+}
+
+// One CTA sorts the pairs by expert. sh: counts [E] (zeroed by the caller) | cursors [E] | tile offsets [E + 1].
 // tiles: [0] = number of tiles, then (expert, first slot) pairs from index 2 on.
-__global__ void __launch_bounds__(1024)
-moe_plan_kernel(const int* __restrict__ sel, int n_pairs, int E, int tile_rows, int* __restrict__ seg_off,
-                int* __restrict__ perm, int* __restrict__ slot_of, int* __restrict__ tiles) {
-    extern __shared__ int sh[];   // counts [E] | cursors [E] | tile offsets [E + 1]
+__device__ __forceinline__ void plan_pairs(const int* __restrict__ sel, int n_pairs, int E, int tile_rows, int* sh,
+                                           int* __restrict__ seg_off, int* __restrict__ perm, int* __restrict__ slot_of,
+                                           int* __restrict__ tiles) {
     int* cnt = sh;
     int* cur = sh + E;
     int* toff = sh + 2 * E;
-    pdl_launch_dependents();
-    for (int e = threadIdx.x; e < E; e += blockDim.x) cnt[e] = 0;
-    pdl_wait();
-    __syncthreads();
     for (int i = threadIdx.x; i < n_pairs; i += blockDim.x) {
         const int e = sel[i];
         if (e >= 0 && e < E) atomicAdd(&cnt[e], 1);
@@ -168,6 +178,34 @@ moe_plan_kernel(const int* __restrict__ sel, int n_pairs, int E, int tile_rows, 
         }
         slot_of[i] = slot;
     }
+}
+
+__global__ void __launch_bounds__(1024)
+moe_plan_kernel(const int* __restrict__ sel, int n_pairs, int E, int tile_rows, int* __restrict__ seg_off,
+                int* __restrict__ perm, int* __restrict__ slot_of, int* __restrict__ tiles) {
+    extern __shared__ int sh[];
+    pdl_launch_dependents();
+    for (int e = threadIdx.x; e < E; e += blockDim.x) sh[e] = 0;
+    pdl_wait();
+    __syncthreads();
+    plan_pairs(sel, n_pairs, E, tile_rows, sh, seg_off, perm, slot_of, tiles);
+}
+
+// Decode-sized steps: routing and plan in one CTA (the choices stay in shared memory on their way to the plan).
+__global__ void __launch_bounds__(1024)
+moe_route_plan_kernel(const __grid_constant__ RouteArgs a, int T, int E, int tile_rows, int* __restrict__ sel,
+                      float* __restrict__ wgt, int* __restrict__ seg_off, int* __restrict__ perm, int* __restrict__ slot_of,
+                      int* __restrict__ tiles) {
+    extern __shared__ int sh[];   // plan_pairs' part [3 E + 1] | choices [T top]
+    int* s_sel = sh + 3 * E + 1;
+    pdl_launch_dependents();
+    for (int e = threadIdx.x; e < E; e += blockDim.x) sh[e] = 0;
+    pdl_wait();
+    for (int t = threadIdx.x >> 5; t < T; t += blockDim.x >> 5) route_token(a, t, s_sel, wgt);
+    __syncthreads();
+    const int n_pairs = T * a.top;
+    for (int i = threadIdx.x; i < n_pairs; i += blockDim.x) sel[i] = s_sel[i];
+    plan_pairs(s_sel, n_pairs, E, tile_rows, sh, seg_off, perm, slot_of, tiles);
 }
 
 constexpr int kET = 64, kEK = 64, kELD = kEK + 8, kEStages = 3;
@@ -489,8 +527,29 @@ int atx_moe_route_scored(const float* logits, long long ld, const float* correct
     cfg.blockDim = dim3(128);
     cfg.stream = reinterpret_cast<cudaStream_t>(stream);
     set_pdl_moe(cfg, attr, flags);
-    ATX_CUDA(cudaLaunchKernelEx(&cfg, moe_route_kernel, logits, ld, correction, R, top, scale, sel, wgt, T, normalize, score,
-                                power));
+    const RouteArgs a{logits, ld, correction, R, top, scale, normalize, score, power};
+    ATX_CUDA(cudaLaunchKernelEx(&cfg, moe_route_kernel, a, sel, wgt, T));
+    return ATX_OK;
+}
+
+int atx_moe_route_plan(const float* logits, long long ld, const float* correction, int R, int top, float scale, int normalize,
+                       int score, int power, int T, int E, int tile_rows, int* sel, float* wgt, int* seg_off, int* perm,
+                       int* slot_of, int* tiles, int flags, atx_stream_t stream) {
+    ATX_REQUIRE(logits && sel && wgt && seg_off && perm && slot_of && tiles, "atx_moe_route_plan: null pointer");
+    ATX_REQUIRE((score == ATX_MOE_SOFTMAX || score == ATX_MOE_SIGMOID) && (power == 1 || power == 2),
+                "atx_moe_route_plan: score=%d power=%d", score, power);
+    ATX_REQUIRE(T > 0 && T <= 64 && R > 0 && R <= 32 * kRouteMax && top > 0 && top <= R && top <= 64 && ld >= R && E > 0 && E <= R &&
+                    tile_rows > 0,
+                "atx_moe_route_plan: bad shape T=%d (<= 64) outputs=%d (<= %d) top=%d ld=%lld experts=%d", T, R, 32 * kRouteMax, top, ld, E);
+    cudaLaunchConfig_t cfg = {};
+    cudaLaunchAttribute attr[1];
+    cfg.gridDim = dim3(1);
+    cfg.blockDim = dim3(T <= 8 ? 256 : 1024);
+    cfg.dynamicSmemBytes = sizeof(int) * (3 * static_cast<size_t>(E) + 1 + static_cast<size_t>(T) * top);
+    cfg.stream = reinterpret_cast<cudaStream_t>(stream);
+    set_pdl_moe(cfg, attr, flags);
+    const RouteArgs a{logits, ld, correction, R, top, scale, normalize, score, power};
+    ATX_CUDA(cudaLaunchKernelEx(&cfg, moe_route_plan_kernel, a, T, E, tile_rows, sel, wgt, seg_off, perm, slot_of, tiles));
     return ATX_OK;
 }
 

@@ -604,6 +604,16 @@ int atx_conv_dt_inplace(const float* in, long long ld, int x_off, int dt_off, co
 #define ATX_MOE_SIGMOID 1
 int atx_moe_route_scored(const float* logits, long long ld, const float* correction, int R, int top, float scale,
                          int normalize, int score, int power, int* sel, float* wgt, int T, int flags, atx_stream_t stream);
+/* atx_moe_route_scored and atx_moe_plan in one launch, for steps of at most 64 tokens (the choices below E are real experts). */
+int atx_moe_route_plan(const float* logits, long long ld, const float* correction, int R, int top, float scale, int normalize,
+                       int score, int power, int T, int E, int tile_rows, int* sel, float* wgt, int* seg_off, int* perm,
+                       int* slot_of, int* tiles, int flags, atx_stream_t stream);
+/* atx_gemm_run_grouped for steps of at most 64 tokens, on the weight-streaming kernel: one tile per chosen group (a plan made with
+ * tile_rows >= 64), n_group rows of W each. perm == NULL: X holds the groups' rows back to back (row = slot). perm != NULL: X
+ * holds the step's T tokens as they are (no gather); out[slot, :] = X[perm[slot] / top, :] W_e^T for the slots of every group. K
+ * is split over a cluster where one wave has room. Modes STORE_F32, STORE_BF16, RELU2_BF16. */
+int atx_gemm_run_grouped_small(const atx_gemm_plan* plan, void* out, long long ldo, int n_group, int mode, const int* seg_off,
+                               const int* tiles, int max_tiles, const int* perm, int top, int T, int flags, atx_stream_t stream);
 /* x[t, n] = cap tanh(x[t, n] / cap) in place, n < N. */
 int atx_soft_cap(float* x, long long ld, int T, int N, float cap, int flags, atx_stream_t stream);
 
