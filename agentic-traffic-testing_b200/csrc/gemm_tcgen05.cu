@@ -925,7 +925,9 @@ int atx_gemm_run(const atx_gemm_plan* p, void* out, long long ldo, int T, int mo
     if (T <= 64) return launch_gemm<64>(p, 2, out, ldo, T, kmode, splits, pdl, stream);
     // prefill-sized batches: the persistent, warp-specialised kernel (one CTA per SM, two TMEM accumulators)
     ATX_REQUIRE(splits == 1, "atx_gemm_run: split-K is for decode-sized steps (T <= 64); got T=%d splits=%d", T, splits);
-    if (T <= 128) return launch_gemm_persistent<128>(p, 3, out, ldo, T, mode, pdl, stream);
+    // (narrow outputs, a router's: half-size token tiles where full ones would leave half of the SMs without work)
+    const long long tiles256 = ((p->N + kBM - 1) / kBM) * ((T + 255) / 256);
+    if (T <= 128 || tiles256 * 2 <= num_sms()) return launch_gemm_persistent<128>(p, 3, out, ldo, T, mode, pdl, stream);
     return launch_gemm_persistent<256>(p, 4, out, ldo, T, mode, pdl, stream);
 }
 

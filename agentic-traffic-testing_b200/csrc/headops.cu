@@ -368,20 +368,45 @@ conv_head_prepare_kernel(const __grid_constant__ ConvPrepArgs a) {
             }
         }
     };
-    float win[NW][E], cur[E], nxt[E];
+    // What the rows of the tile belong to, a row per lane; the angles of a row and its projection are fetched one row ahead.
+    int m_seq = -1, m_slot = -1, m_pos = 0;
+    if (lane < a.rows_per && t0 + lane < a.T) m_seq = a.tok_seq[t0 + lane], m_slot = a.slots[t0 + lane], m_pos = a.positions[t0 + lane];
+    constexpr int NP = E / 2;   // rotated pairs of a lane
+    float win[NW][E], cur[E], nxt[E], cn[NP], sn[NP], cx[NP], sx[NP];
+    auto angles = [&](int pos) {
+        const float* cs = s.rot + static_cast<long long>(pos) * s.rot_dims;
+#pragma unroll
+        for (int g = 0; g < NG; ++g)
+#pragma unroll
+            for (int e = 0; e < VE; e += 2) {
+                const int p = (el[g] + e) >> 1, q = (g * VE + e) >> 1;
+                cx[q] = p < half ? cs[p] : 1.f;
+                sx[q] = p < half ? cs[half + p] : 0.f;
+            }
+    };
     load(a.src + static_cast<long long>(t0) * a.ld + col, nxt);
+    if (half > 0) angles(__shfl_sync(0xffffffffu, m_pos, 0));
     int prev_s = -1, prev_i = -2;
+    float* st = nullptr;
     for (int r = 0; r < a.rows_per && t0 + r < a.T; ++r) {
         const long long t = t0 + r;
 #pragma unroll
         for (int e = 0; e < E; ++e) cur[e] = nxt[e];
-        if (r + 1 < a.rows_per && t + 1 < a.T) load(a.src + (t + 1) * a.ld + col, nxt);   // the next row while this one is worked on
-        const int sq = a.tok_seq[t], slot = a.slots[t];
-        if (sq < 0 || slot < 0) continue;   // padded row
-        const int i = static_cast<int>(t) - a.seq_start[sq];
-        float* st = a.conv_state + static_cast<long long>(a.seq_slot[sq]) * (K - 1) * a.C + ch;
-        if (sq != prev_s || i != prev_i + 1) {
+#pragma unroll
+        for (int q = 0; q < NP; ++q) cn[q] = cx[q], sn[q] = sx[q];
+        const int sq = __shfl_sync(0xffffffffu, m_seq, r), slot = __shfl_sync(0xffffffffu, m_slot, r);
+        if (r + 1 < a.rows_per && t + 1 < a.T) {
+            load(a.src + (t + 1) * a.ld + col, nxt);
+            if (half > 0) angles(__shfl_sync(0xffffffffu, m_pos, r + 1));
+        }
+        if (sq < 0 || slot < 0) {   // padded row
+            prev_s = -1;
+            continue;
+        }
+        const int i = sq == prev_s ? prev_i + 1 : static_cast<int>(t) - a.seq_start[sq];   // a sequence's rows are consecutive
+        if (sq != prev_s) {
             const int pos0 = a.seq_pos0[sq];
+            st = a.conv_state + static_cast<long long>(a.seq_slot[sq]) * (K - 1) * a.C + ch;
 #pragma unroll
             for (int j = 0; j < NW; ++j) {
 #pragma unroll
@@ -440,18 +465,12 @@ conv_head_prepare_kernel(const __grid_constant__ ConvPrepArgs a) {
         const long long page = ((static_cast<long long>(blk) * s.heads + hh) * a.bs + off) * width;
         if (s.raw_dst) put(reinterpret_cast<XT*>(s.raw_dst) + page, u);
         if (half > 0) {
-            const float* cs = s.rot + static_cast<long long>(a.positions[t]) * s.rot_dims;
 #pragma unroll
-            for (int g = 0; g < NG; ++g)
-#pragma unroll
-                for (int e = 0; e < VE; e += 2) {
-                    const int p = (el[g] + e) >> 1;
-                    if (p < half) {
-                        const float c = cs[p], sn = cs[half + p], x = u[g * VE + e], y = u[g * VE + e + 1];
-                        u[g * VE + e] = fmaf(x, c, -(y * sn));
-                        u[g * VE + e + 1] = fmaf(y, c, x * sn);
-                    }
-                }
+            for (int q = 0; q < NP; ++q) {   // pairs past the rotated range carry the angle 0
+                const float x = u[2 * q], y = u[2 * q + 1];
+                u[2 * q] = fmaf(x, cn[q], -(y * sn[q]));
+                u[2 * q + 1] = fmaf(y, cn[q], x * sn[q]);
+            }
         }
         if (s.norm) {
             float ss = 0.f;

@@ -232,7 +232,7 @@ __device__ __forceinline__ float row_sum(float v, float* red) {   // over the CT
 }
 
 template <typename XT, int NV>
-__global__ void __launch_bounds__(1024)
+__global__ void __launch_bounds__(NV == 8 ? 512 : 1024)
 parallel_resid_norm_kernel(const __grid_constant__ ParallelResidArgs a) {
     extern __shared__ __align__(16) float srow_p[];
     __shared__ float red[32];
