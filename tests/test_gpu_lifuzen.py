@@ -268,7 +268,7 @@ def tc_model(all_experts=False):
     top = lambda e, t: e if all_experts else t
     return model_cfg([mamba(heads=4, vdim=64, state=64, groups=2, norm_groups=2, conv=4, mlp=moe(4, top(4, 2), 64)),
                       att(heads=4, kv=2, dim=64, dims=32, scale=0.125, mlp=moe(6, top(6, 1), 128)),
-                      att(heads=2, kv=1, dim=128, dims=128, base=20000.0, scale=0.09, conv=3, mlp=moe(2, 2, 64)),
+                      att(heads=2, kv=1, dim=128, dims=128, base=15000.0, scale=0.09, conv=3, mlp=moe(2, 2, 64)),
                       mamba(heads=2, vdim=96, state=32, groups=1, norm_groups=1, conv=2),
                       att(heads=8, kv=1, dim=40, dims=16, scale=0.15, conv=2)], width=128, loop=(1, 3, 2))
 
