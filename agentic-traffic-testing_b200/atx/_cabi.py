@@ -22,6 +22,8 @@ GEMM_SWIGLU_BF16 = 3
 GEMM_RELU2_BF16 = 4
 GEMM_GLU_CLAMP_BF16 = 5
 GEMM_SOFTCAP_F32 = 6
+GEMM_GEGLU_BF16 = 7
+GEMM_GATED = (GEMM_SWIGLU_BF16, GEMM_GLU_CLAMP_BF16, GEMM_GEGLU_BF16)   # W holds gate and up rows, the output N / 2 columns
 FLAG_PDL = 1
 FLAG_ORDERED = 2   # atx_gemm_run ADD_F32, T <= 64: fixed-order split-K (bit-reproducible)
 FLAG_ADD_BF16 = 4  # atx_rmsnorm: the `add` buffer is bf16
@@ -53,11 +55,14 @@ EXPORTS = [
     "atx_gated_linear_recurrence_chunked", "atx_gated_linear_recurrence_chunked_supported",
     "atx_parallel_resid_norm", "atx_conv_head_prepare", "atx_conv_dt_inplace", "atx_moe_route_scored", "atx_soft_cap",
     "atx_moe_route_plan", "atx_gemm_run_grouped_small",
+    "atx_qk_prepare_temp", "atx_linear_recurrence_rot", "atx_linear_recurrence_rot_chunked", "atx_gated_act_kind",
+    "atx_moe_route_biased", "atx_moe_route_plan_biased",
 ]
 ATTN_SOFTMAX = 0
 ATTN_SIGMOID = 1
 ACT_RELU2 = 0
 ACT_GELU_TANH = 1
+ACT_SILU = 2
 HEAD_DST_ROWS = 0
 HEAD_DST_PAGES = 1
 HEAD_SEGS_MAX = 4
@@ -92,7 +97,8 @@ class ResidTerms(C.Structure):
 
     _fields_ = [("y", C.c_void_p), ("experts", C.c_void_p), ("wgt", C.c_void_p), ("slot_of", C.c_void_p), ("ids", C.c_void_p),
                 ("table", C.c_void_p), ("vec", C.c_void_p), ("lde", C.c_longlong), ("y_scale", C.c_float),
-                ("zero_y", C.c_int), ("top", C.c_int), ("vocab", C.c_int), ("table_mode", C.c_int)]
+                ("zero_y", C.c_int), ("top", C.c_int), ("vocab", C.c_int), ("table_mode", C.c_int),
+                ("table_w", C.c_void_p)]
 
 
 class AttnOpts(C.Structure):
@@ -245,6 +251,15 @@ def load() -> C.CDLL:
     lib.atx_moe_route_plan.argtypes = [vp, i64, vp, i32, i32, f32, i32, i32, i32, i32, i32, i32, vp, vp, vp, vp, vp, vp, i32, vp]
     lib.atx_gemm_run_grouped_small.argtypes = [vp, vp, i64, i32, i32, vp, vp, i32, vp, i32, i32, i32, vp]
     lib.atx_soft_cap.argtypes = [vp, i64, i32, i32, f32, i32, vp]
+    lib.atx_qk_prepare_temp.argtypes = [vp, i64, i32, i32, i32, vp, vp, vp, vp, vp, vp, i32, f32, f32, vp, vp, vp, vp, vp, i32, i32,
+                                        i32, i32, i32, i32, f32, i32, i32, vp]
+    lib.atx_linear_recurrence_rot.argtypes = [vp, i64, vp, i64, vp, i64, i32, i32, i32, i32, vp, vp, vp, vp, i32, vp, i32, f32, vp,
+                                              vp, i64, vp, vp, vp, vp, i32, i32, vp]
+    lib.atx_linear_recurrence_rot_chunked.argtypes = list(lib.atx_linear_recurrence_rot.argtypes)
+    lib.atx_gated_act_kind.argtypes = [vp, vp, i32, i32, i32, i32, i32, vp]
+    lib.atx_moe_route_biased.argtypes = [vp, i64, vp, vp, i32, i32, f32, i32, i32, i32, vp, vp, i32, i32, vp]
+    lib.atx_moe_route_plan_biased.argtypes = [vp, i64, vp, vp, i32, i32, f32, i32, i32, i32, i32, i32, i32, vp, vp, vp, vp, vp, vp,
+                                              i32, vp]
     for name in EXPORTS:  # fail at load time, not at first use, if the build is stale
         getattr(lib, name)
     _lib = lib
@@ -291,8 +306,8 @@ class GemmPlan:
 
     def run(self, out: torch.Tensor, T: int, mode: int, splits: int = 0, flags: int = 0) -> None:
         _dev(out)
-        want = torch.bfloat16 if mode in (GEMM_STORE_BF16, GEMM_SWIGLU_BF16, GEMM_RELU2_BF16, GEMM_GLU_CLAMP_BF16) else torch.float32
-        cols = self.N // 2 if mode in (GEMM_SWIGLU_BF16, GEMM_GLU_CLAMP_BF16) else self.N
+        want = torch.bfloat16 if mode in (GEMM_STORE_BF16, GEMM_RELU2_BF16) + GEMM_GATED else torch.float32
+        cols = self.N // 2 if mode in GEMM_GATED else self.N
         assert out.dtype == want and out.dim() == 2 and out.shape[1] >= cols and out.shape[0] >= T
         _check(load().atx_gemm_run(self._h, out.data_ptr(), out.stride(0), T, mode, splits, flags, _stream()))
 

@@ -10,9 +10,10 @@ from typing import Optional
 
 
 def _entries():
-    from . import gopopel, lifuzen, napuzen, safisun, zonidra
+    from . import gopopel, lifuzen, napuzen, safisun, sutosun, zonidra
 
-    return {"safisun": safisun, "gopopel": gopopel, "zonidra": zonidra, "napuzen": napuzen, "lifuzen": lifuzen}
+    return {"safisun": safisun, "gopopel": gopopel, "zonidra": zonidra, "napuzen": napuzen, "lifuzen": lifuzen,
+            "sutosun": sutosun}
 
 
 def _module(arch: str):

@@ -40,7 +40,7 @@ from typing import Dict, List, Optional, Tuple
 import torch
 
 from .. import _cabi
-from .common import UngatedExperts, _Linear, rotation_table
+from .common import Experts, PagedAttention, _Linear, rotation_table
 
 MIXERS = ("mamba2", "attention")
 NORM_SHIFT = 1.0       # norm weights are stored around zero
@@ -398,7 +398,8 @@ class Program:
         self.q_flat = torch.zeros(T * n_q, dtype=xt, device=dev)
         self.mix_flat = torch.zeros(T * n_mix, dtype=xt, device=dev)
         self.xl = torch.zeros(r.Rmax, W, dtype=xt, device=dev)
-        self.experts = UngatedExperts(lib, r._ck, [s["mlp"] for s in cfg.layers if s.get("mlp") is not None], T, W, self.xf, self.dt)
+        # (squared scores: the weight multiplies the input of an expert of degree two)
+        self.experts = Experts(lib, r._ck, [s["mlp"] for s in cfg.layers if s.get("mlp") is not None], T, W, self.xf, self.dt, power=2)
         self._views: Dict[Tuple[int, int], torch.Tensor] = {}
 
         def view(flat: torch.Tensor, k: int) -> torch.Tensor:
@@ -455,11 +456,7 @@ class Program:
         self.overlap_ffn = True
         self.side = torch.cuda.Stream(device=dev)
         self.ev_fork, self.ev_join = torch.cuda.Event(), torch.cuda.Event()
-        # scratch of the decode attention's key slices: [tokens, heads, slices, value width + 2] fp32
-        self.max_splits = 32
-        self.sms = torch.cuda.get_device_properties(dev).multi_processor_count
-        h_max = max(int(s["mixer"]["heads"]) for s in cfg.layers)
-        self.split_ws = torch.zeros(max(2, S * h_max * self.max_splits * (128 + 2)), dtype=f32, device=dev)
+        self.attention = PagedAttention(r, self.dt, max(int(s["mixer"]["heads"]) for s in cfg.layers))
         self._opts: List[Optional[_cabi.AttnOpts]] = []
         for spec in cfg.layers:
             o = None
@@ -475,9 +472,7 @@ class Program:
     def _attention(self, ri: int, li: int, proj: int, ld: int, out: int, ldo: int, T: int, n_dec: int, n_pf: int, fl: int,
                    st: int) -> int:
         """proj columns [q | k] of one layer run: convolution, rotation, norm, page write, then attention of the step's rows over
-        their sequences' pages. Prompt portions on the tensor cores where the element type and the sizes have such a kernel;
-        single decoded tokens (and every row otherwise) on the decode form of that kernel or on the kernel that gives a warp
-        to each (row, head). Returns the launch count."""
+        their sequences' pages. Returns the launch count."""
         r, lib, ck, dp, dt = self.r, self.r.lib, self.r._ck, self.r._dp, self.dt
         c, l = self.cfg.layers[li]["mixer"], self.w.layers[li]
         H, G, D, K = (int(c[k]) for k in ("heads", "kv_heads", "dim", "conv"))
@@ -498,26 +493,7 @@ class Program:
             ck(lib.atx_conv_state_update(proj, ld, 0, cs, *(dp[k] + 4 * n_dec for k in ("seq_start", "seq_count", "seq_pos0", "seq_slot")),
                                          n_pf, C, K, fl, st))
             n += 1
-        po = ctypes.byref(self._opts[li])
-        tc = n_pf > 0 and lib.atx_attn_window_prefill_supported(D, D, D, D, dt)
-        rows = n_dec if tc else T
-        if rows and rows == n_dec and lib.atx_attn_window_decode_supported(H, G, D, D, D, D, dt):
-            splits = max(1, min((r.e.max_model_len + 63) // 64, self.max_splits, -(-3 * self.sms // (rows * G))))
-            ws = self.split_ws
-            ck(lib.atx_attn_paged_decode(q, kc, vc, D, D, dp["seq_bt"], r.MB, dp["tok_seq"], dp["pos"], None, 0, out, ldo,
-                                         ws.data_ptr(), ws.numel() * 4, splits, rows, H, G, D, D, r.bs, po, dt, fl, st))
-            n += 2 if splits > 1 else 1
-        elif rows:
-            ck(lib.atx_attn_paged(q, kc, vc, D, D, dp["seq_bt"], r.MB, dp["tok_seq"], dp["pos"], None, 0, out, ldo, rows, H, G,
-                                  D, D, r.bs, po, dt, fl, st))
-            n += 1
-        if tc:
-            # rows of the prompt portions start at row n_dec: q and out are passed whole, rows come from seq_start
-            ck(lib.atx_attn_paged_prefill(q, kc, vc, D, D, dp["seq_bt"] + 4 * n_dec * r.MB, r.MB, dp["seq_start"] + 4 * n_dec,
-                                          dp["seq_count"] + 4 * n_dec, dp["seq_pos0"] + 4 * n_dec, n_pf, T - n_dec, None, 0,
-                                          out, ldo, H, G, D, D, r.bs, po, dt, fl, st))
-            n += 1
-        return n
+        return n + self.attention.run(self._opts[li], q, kc, vc, D, D, H, G, D, D, None, 0, out, ldo, T, n_dec, n_pf, fl, st)
 
     def _mamba2(self, ri: int, li: int, proj: int, ld: int, out: int, ldo: int, T: int, n_dec: int, n_pf: int, fl: int,
                 st: int) -> int:

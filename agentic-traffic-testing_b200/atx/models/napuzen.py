@@ -45,7 +45,7 @@ from typing import Dict, List, Optional, Tuple
 import torch
 
 from .. import _cabi
-from .common import _Linear, _use_tc, rotation_table_scaled, stretched_frequencies
+from .common import PagedAttention, _Linear, _use_tc, rotation_table_scaled, stretched_frequencies
 
 MIXERS = ("gla", "latent_attention", "latent_attention_2")
 GLU_ALPHA = 1.702      # the dense feed-forward's gate is g * sigmoid(GLU_ALPHA * g) ...
@@ -576,11 +576,8 @@ class Program:
         self.state: List[Optional[torch.Tensor]] = [
             torch.zeros(S, int(sp["mixer"]["heads"]), int(sp["mixer"]["dim"]), int(sp["mixer"]["vdim"]), dtype=f32, device=dev)
             if sp["type"] == "gla" else None for sp in cfg.layers]
-        # scratch of the decode attention's key slices: [tokens, heads, slices, value width + 2] fp32
-        self.max_splits = 32
         self.sms = torch.cuda.get_device_properties(dev).multi_processor_count
-        h_max = max(int(sp["mixer"]["heads"]) for sp in cfg.layers)
-        self.split_ws = torch.zeros(max(2, S * h_max * self.max_splits * (128 + 2)), dtype=f32, device=dev)
+        self.attention = PagedAttention(r, self.dt, max(int(sp["mixer"]["heads"]) for sp in cfg.layers))
         self._opts: List[Optional[_cabi.AttnOpts]] = []
         for spec in cfg.layers:
             c = spec["mixer"]
@@ -598,38 +595,11 @@ class Program:
     def _attend(self, li: int, q: int, row: int, Dk: int, Vd: int, gate, ldg: int, out: int, ldo: int, T: int, n_dec: int,
                 n_pf: int) -> int:
         """Attention of the step's rows over their sequences' latent pages (one key/value head of `row` elements shared by
-        all query heads; the key is the row's first Dk elements, the value its first Vd): prompt portions on the tensor
-        cores where the element type and the sizes have such a kernel; single decoded tokens (and every row otherwise) on
-        the decode form of that kernel or on the kernel that gives a warp to each (row, head). Returns the launch count."""
-        import ctypes
-
-        r, lib, ck, dp, dt = self.r, self.r.lib, self.r._ck, self.r._dp, self.dt
+        all query heads; the key is the row's first Dk elements, the value its first Vd). Returns the launch count."""
         H = int(self.cfg.layers[li]["mixer"]["heads"])
         kc = self.pages[li].data_ptr()
-        o = self._opts[li]
-        po = ctypes.byref(o)
-        fl, st = r.flags, torch.cuda.current_stream().cuda_stream
-        tc = n_pf > 0 and lib.atx_attn_window_prefill_supported(Dk, Vd, row, row, dt)
-        rows = n_dec if tc else T
-        n = 0
-        if rows and rows == n_dec and lib.atx_attn_window_decode_supported(H, 1, Dk, Vd, row, row, dt):
-            keys = min(o.window if o.window else r.e.max_model_len, r.e.max_model_len)
-            splits = max(1, min((keys + 63) // 64, self.max_splits, -(-3 * self.sms // rows)))
-            ws = self.split_ws
-            ck(lib.atx_attn_paged_decode(q, kc, kc, row, row, dp["seq_bt"], r.MB, dp["tok_seq"], dp["pos"], gate, ldg, out, ldo,
-                                         ws.data_ptr(), ws.numel() * 4, splits, rows, H, 1, Dk, Vd, r.bs, po, dt, fl, st))
-            n += 2 if splits > 1 else 1
-        elif rows:
-            ck(lib.atx_attn_paged(q, kc, kc, row, row, dp["seq_bt"], r.MB, dp["tok_seq"], dp["pos"], gate, ldg, out, ldo, rows, H,
-                                  1, Dk, Vd, r.bs, po, dt, fl, st))
-            n += 1
-        if tc:
-            # rows of the prompt portions start at row n_dec: q, gate and out are passed whole, rows come from seq_start
-            ck(lib.atx_attn_paged_prefill(q, kc, kc, row, row, dp["seq_bt"] + 4 * n_dec * r.MB, r.MB, dp["seq_start"] + 4 * n_dec,
-                                          dp["seq_count"] + 4 * n_dec, dp["seq_pos0"] + 4 * n_dec, n_pf, T - n_dec, gate, ldg,
-                                          out, ldo, H, 1, Dk, Vd, r.bs, po, dt, fl, st))
-            n += 1
-        return n
+        return self.attention.run(self._opts[li], q, kc, kc, row, row, H, 1, Dk, Vd, gate, ldg, out, ldo, T, n_dec, n_pf, self.r.flags,
+                                  torch.cuda.current_stream().cuda_stream)
 
     def forward(self, T: int, n_dec: int, n_pf: int, n_rows: int) -> int:
         """Issue every kernel of one step on the current stream; returns the launch count. The step's first n_dec

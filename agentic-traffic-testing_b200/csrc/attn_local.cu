@@ -1,5 +1,5 @@
 // Softmax attention over the paged KV cache with the options the Llama path does not have: biases on q/k/v, an RMS norm
-// over the whole q (and k) projection, rotation of the first `rot_dims` dimensions of a head in adjacent pairs,
+// over the whole q (and k) projection, a query factor that grows with the position, rotation of the first `rot_dims` dimensions of a head in adjacent pairs,
 // a tanh cap on the scores, a block-local causal mask (a query sees the keys of its own block of `chunk` positions),
 // a zero-score sink in the softmax denominator, a sigmoid gate per head on the output, any head sizes (the value size
 // may differ from the query/key size); and, each optional: a sliding window, a penalty per head and unit of distance,
@@ -36,14 +36,16 @@ __device__ __forceinline__ void stx2(__nv_bfloat16* p, long long i, float a, flo
 }
 
 // ---- bias, whole-projection RMS norm, partial rotation, page scatter ----------------------------------------------
-// One block per row. rot: [max_pos, rot_dims] fp32, cos of the rot_dims/2 angles then their sines.
+// One block per row. rot: [max_pos, rot_dims] fp32, cos of the rot_dims/2 angles then their sines. qt_coef != 0: the query at
+// position p is multiplied by 1 + qt_coef ln(floor((p + 1) / qt_every) + 1).
 template <typename XT>
 __global__ void __launch_bounds__(256)
 qk_prepare_kernel(const float* __restrict__ proj, long long ld, int q_off, int k_off, int v_off,
                   const XT* __restrict__ bq, const XT* __restrict__ bk, const XT* __restrict__ bv,
                   const XT* __restrict__ wq, const XT* __restrict__ wk, const float* __restrict__ rot, int rot_dims,
                   const int* __restrict__ positions, const int* __restrict__ slots, XT* __restrict__ q_out,
-                  XT* __restrict__ k_cache, XT* __restrict__ v_cache, int H, int G, int D, int Vd, int bs, float eps) {
+                  XT* __restrict__ k_cache, XT* __restrict__ v_cache, int H, int G, int D, int Vd, int bs, float eps,
+                  float qt_coef, float qt_every) {
     extern __shared__ float sm[];
     __shared__ float red[2][32];
     pdl_launch_dependents();
@@ -108,9 +110,10 @@ qk_prepare_kernel(const float* __restrict__ proj, long long ld, int q_off, int k
         tq += red[0][i];
         tk += red[1][i];
     }
-    const float rq = wq ? rsqrtf(tq / static_cast<float>(nq) + eps) : 1.f;
-    const float rk = wk ? rsqrtf(tk / static_cast<float>(nk) + eps) : 1.f;
     const int pos = positions[t];
+    float rq = wq ? rsqrtf(tq / static_cast<float>(nq) + eps) : 1.f;
+    const float rk = wk ? rsqrtf(tk / static_cast<float>(nk) + eps) : 1.f;
+    if (qt_coef != 0.f) rq *= fmaf(qt_coef, logf(floorf(static_cast<float>(pos + 1) / qt_every) + 1.f), 1.f);
     const float* cs = rot + static_cast<long long>(pos) * rot_dims;
     const int half = rot_dims / 2;
     const int blk = slot / bs, off = slot - blk * bs;
@@ -742,7 +745,17 @@ int atx_qk_prepare(const float* proj, long long ld, int q_off, int k_off, int v_
                    const void* bv, const void* wq, const void* wk, const float* rot, int rot_dims, const int* positions,
                    const int* slots, void* q_out, void* k_cache, void* v_cache, int T, int H, int G, int D, int Vd,
                    int block_size, float eps, int dtype, int flags, atx_stream_t stream) {
+    return atx_qk_prepare_temp(proj, ld, q_off, k_off, v_off, bq, bk, bv, wq, wk, rot, rot_dims, 0.f, 1.f, positions, slots, q_out,
+                               k_cache, v_cache, T, H, G, D, Vd, block_size, eps, dtype, flags, stream);
+}
+
+int atx_qk_prepare_temp(const float* proj, long long ld, int q_off, int k_off, int v_off, const void* bq, const void* bk,
+                        const void* bv, const void* wq, const void* wk, const float* rot, int rot_dims, float qt_coef,
+                        float qt_every, const int* positions, const int* slots, void* q_out, void* k_cache, void* v_cache,
+                        int T, int H, int G, int D, int Vd, int block_size, float eps, int dtype, int flags,
+                        atx_stream_t stream) {
     ATX_REQUIRE(proj && positions && slots && q_out && k_cache && v_cache, "atx_qk_prepare: null pointer");
+    ATX_REQUIRE(qt_every > 0.f, "atx_qk_prepare: qt_every=%g must be positive", qt_every);
     ATX_REQUIRE(T > 0 && H > 0 && G > 0 && H % G == 0 && D > 0 && D % 2 == 0 && Vd > 0 && block_size > 0,
                 "atx_qk_prepare: bad shape T=%d H=%d G=%d D=%d Vd=%d", T, H, G, D, Vd);
     ATX_REQUIRE(rot_dims >= 0 && rot_dims % 2 == 0 && rot_dims <= D && (rot_dims == 0 || rot),
@@ -770,7 +783,7 @@ int atx_qk_prepare(const float* proj, long long ld, int q_off, int k_off, int v_
                                     reinterpret_cast<const float*>(bv), reinterpret_cast<const float*>(wq),
                                     reinterpret_cast<const float*>(wk), rot, rot_dims, positions, slots,
                                     reinterpret_cast<float*>(q_out), reinterpret_cast<float*>(k_cache),
-                                    reinterpret_cast<float*>(v_cache), H, G, D, Vd, block_size, eps));
+                                    reinterpret_cast<float*>(v_cache), H, G, D, Vd, block_size, eps, qt_coef, qt_every));
     } else {
         using B = __nv_bfloat16;
         if (smem > 48 * 1024)
@@ -781,7 +794,7 @@ int atx_qk_prepare(const float* proj, long long ld, int q_off, int k_off, int v_
                                     reinterpret_cast<const B*>(bv), reinterpret_cast<const B*>(wq),
                                     reinterpret_cast<const B*>(wk), rot, rot_dims, positions, slots,
                                     reinterpret_cast<B*>(q_out), reinterpret_cast<B*>(k_cache),
-                                    reinterpret_cast<B*>(v_cache), H, G, D, Vd, block_size, eps));
+                                    reinterpret_cast<B*>(v_cache), H, G, D, Vd, block_size, eps, qt_coef, qt_every));
     }
     return ATX_OK;
 }

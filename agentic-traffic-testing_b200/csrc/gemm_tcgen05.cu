@@ -25,16 +25,19 @@
 namespace atx {
 
 // The gated epilogues: ATX_GEMM_SWIGLU_BF16 = silu(gate) * up; ATX_GEMM_GLU_CLAMP_BF16 = g sigmoid(alpha g) (u + shift) with
-// g = min(gate, limit), u = clamp(up, -limit, limit) (alpha, limit, shift: atx_gemm_plan_set_gate). Same tile layout.
+// g = min(gate, limit), u = clamp(up, -limit, limit) (alpha, limit, shift: atx_gemm_plan_set_gate); ATX_GEMM_GEGLU_BF16 =
+// gelu(gate) * up in the tanh form of gelu. Same tile layout.
 // ATX_GEMM_SOFTCAP_F32 = limit tanh(acc / limit), stored as fp32 (the cap on a model's logits).
 struct GateParams {
     float alpha, limit, shift;
 };
 __host__ __device__ __forceinline__ bool is_glu(int mode) {
-    return mode == ATX_GEMM_SWIGLU_BF16 || mode == ATX_GEMM_GLU_CLAMP_BF16;
+    return mode == ATX_GEMM_SWIGLU_BF16 || mode == ATX_GEMM_GLU_CLAMP_BF16 || mode == ATX_GEMM_GEGLU_BF16;
 }
 __device__ __forceinline__ float glu_value(float g, float u, int mode, const GateParams& gp) {
     if (mode == ATX_GEMM_SWIGLU_BF16) return g / (1.f + expf(-g)) * u;
+    if (mode == ATX_GEMM_GEGLU_BF16)   // (1 + tanh x) / 2 = 1 / (1 + exp(-2 x))
+        return g / (1.f + expf(-1.5957691216057308f * (g + 0.044715f * g * g * g))) * u;
     g = fminf(g, gp.limit);
     u = fminf(fmaxf(u, -gp.limit), gp.limit);
     return g / (1.f + expf(-gp.alpha * g)) * (u + gp.shift);
@@ -312,8 +315,10 @@ gemm_wt_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
                         const int t = t0 + c + j;
                         const float mine = __uint_as_float(v[j]), other = sx[(c + j) * 64 + i];
                         const float g = gate_warp ? mine : other, u = gate_warp ? other : mine;
-                        if (ok && t < T)
-                            o[static_cast<long long>(t) * ldo + col] = __float2bfloat16_rn(glu_value(g, u, mode, gate_params));
+                        if (!ok || t >= T) continue;
+                        const int orow = by_token ? s_row[c + j] : t;
+                        if (orow >= 0)
+                            o[static_cast<long long>(orow) * ldo + col] = __float2bfloat16_rn(glu_value(g, u, mode, gate_params));
                     }
                 }
             }
@@ -891,7 +896,7 @@ int atx_gemm_run(const atx_gemm_plan* p, void* out, long long ldo, int T, int mo
     cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_);
     ATX_REQUIRE(p && out, "atx_gemm_run: null pointer");
     ATX_REQUIRE(T > 0 && T <= p->T_cap, "atx_gemm_run: T=%d outside (0, %lld]", T, p->T_cap);
-    ATX_REQUIRE(mode >= ATX_GEMM_STORE_F32 && mode <= ATX_GEMM_SOFTCAP_F32, "atx_gemm_run: bad mode %d", mode);
+    ATX_REQUIRE(mode >= ATX_GEMM_STORE_F32 && mode <= ATX_GEMM_GEGLU_BF16, "atx_gemm_run: bad mode %d", mode);
     ATX_REQUIRE(ldo >= (is_glu(mode) ? p->N / 2 : p->N), "atx_gemm_run: ldo=%lld too small for N=%lld", ldo, p->N);
     ATX_REQUIRE(!is_glu(mode) || p->N % 128 == 0, "atx_gemm_run: SWIGLU mode needs N %% 128 == 0");
     // ATX_FLAG_ORDERED: the K-splits of an ADD are reduced inside a cluster in a fixed order (as for SwiGLU) and ONE CTA
@@ -955,10 +960,11 @@ int atx_gemm_run_grouped_small(const atx_gemm_plan* p, void* out, long long ldo,
     ATX_REQUIRE(p && out && seg_off && tiles, "atx_gemm_run_grouped_small: null pointer");
     ATX_REQUIRE(T > 0 && T <= 64 && max_tiles > 0 && max_tiles <= 65535 && top > 0, "atx_gemm_run_grouped_small: T=%d (1..64) tiles=%d", T,
                 max_tiles);
-    ATX_REQUIRE(n_group > 0 && p->N % n_group == 0 && ldo >= n_group,
+    ATX_REQUIRE(n_group > 0 && p->N % n_group == 0 && ldo >= (is_glu(mode) ? n_group / 2 : n_group),
                 "atx_gemm_run_grouped_small: W has %lld rows, not a multiple of %d per group (ldo=%lld)", p->N, n_group, ldo);
-    ATX_REQUIRE(mode == ATX_GEMM_STORE_F32 || mode == ATX_GEMM_STORE_BF16 || mode == ATX_GEMM_RELU2_BF16,
-                "atx_gemm_run_grouped_small: mode %d (plain stores and the squared ReLU)", mode);
+    ATX_REQUIRE(mode == ATX_GEMM_STORE_F32 || mode == ATX_GEMM_STORE_BF16 || mode == ATX_GEMM_RELU2_BF16 ||
+                    (is_glu(mode) && n_group % 128 == 0),
+                "atx_gemm_run_grouped_small: mode %d (plain stores, the squared ReLU, gated forms over groups of 128 j rows)", mode);
     // K-splits of a tile are a cluster whose leader sums them in a fixed order: as many as still fit one wave of two CTAs per SM
     const long long ctas = static_cast<long long>((n_group + kBM - 1) / kBM) * max_tiles;
     const int kb = static_cast<int>(p->K / kBK);

@@ -1,6 +1,6 @@
 // Mixture of experts: routing, the plan that sorts (token, choice) pairs by expert, the experts' matrix products over
 // their own rows, and the weighted sum.
-//   route    soft-max over the router's outputs, or a sigmoid of each, in fp32; the `top` largest of score + correction are
+//   route    soft-max over the router's outputs (plus a bias per output, if given), or a sigmoid of each, in fp32; the `top` largest of score + correction are
 //            chosen (lowest index on ties), their weight is the plain score times a constant. One warp per token.
 //   plan     one CTA: rows per expert, their running offsets, a slot in the sorted order for every pair whose choice is a
 //            real expert (choices >= E stand for experts that return their input and take no slot), and the list of
@@ -49,6 +49,7 @@ struct RouteArgs {
     int R, top;
     float scale;
     int normalize, score, power;
+    const float* bias;   // added to the logits (nullable)
 };
 
 // One warp routes token t.
@@ -62,7 +63,7 @@ __device__ __forceinline__ void route_token(const RouteArgs& a, long long t, int
 #pragma unroll
     for (int i = 0; i < kRouteMax; ++i) {
         const int e = lane + 32 * i;
-        s[i] = e < R ? z[e] : -INFINITY;
+        s[i] = e < R ? z[e] + (a.bias ? a.bias[e] : 0.f) : -INFINITY;
         mx = fmaxf(mx, s[i]);
     }
     if (score == ATX_MOE_SIGMOID) {
@@ -516,6 +517,12 @@ int atx_moe_route_opts(const float* logits, long long ld, const float* correctio
 
 int atx_moe_route_scored(const float* logits, long long ld, const float* correction, int R, int top, float scale,
                          int normalize, int score, int power, int* sel, float* wgt, int T, int flags, atx_stream_t stream) {
+    return atx_moe_route_biased(logits, ld, nullptr, correction, R, top, scale, normalize, score, power, sel, wgt, T, flags, stream);
+}
+
+int atx_moe_route_biased(const float* logits, long long ld, const float* bias, const float* correction, int R, int top,
+                         float scale, int normalize, int score, int power, int* sel, float* wgt, int T, int flags,
+                         atx_stream_t stream) {
     ATX_REQUIRE((score == ATX_MOE_SOFTMAX || score == ATX_MOE_SIGMOID) && (power == 1 || power == 2),
                 "atx_moe_route: score=%d power=%d", score, power);
     ATX_REQUIRE(logits && sel && wgt, "atx_moe_route: null pointer");
@@ -527,7 +534,7 @@ int atx_moe_route_scored(const float* logits, long long ld, const float* correct
     cfg.blockDim = dim3(128);
     cfg.stream = reinterpret_cast<cudaStream_t>(stream);
     set_pdl_moe(cfg, attr, flags);
-    const RouteArgs a{logits, ld, correction, R, top, scale, normalize, score, power};
+    const RouteArgs a{logits, ld, correction, R, top, scale, normalize, score, power, bias};
     ATX_CUDA(cudaLaunchKernelEx(&cfg, moe_route_kernel, a, sel, wgt, T));
     return ATX_OK;
 }
@@ -535,6 +542,13 @@ int atx_moe_route_scored(const float* logits, long long ld, const float* correct
 int atx_moe_route_plan(const float* logits, long long ld, const float* correction, int R, int top, float scale, int normalize,
                        int score, int power, int T, int E, int tile_rows, int* sel, float* wgt, int* seg_off, int* perm,
                        int* slot_of, int* tiles, int flags, atx_stream_t stream) {
+    return atx_moe_route_plan_biased(logits, ld, nullptr, correction, R, top, scale, normalize, score, power, T, E, tile_rows, sel,
+                                     wgt, seg_off, perm, slot_of, tiles, flags, stream);
+}
+
+int atx_moe_route_plan_biased(const float* logits, long long ld, const float* bias, const float* correction, int R, int top,
+                              float scale, int normalize, int score, int power, int T, int E, int tile_rows, int* sel,
+                              float* wgt, int* seg_off, int* perm, int* slot_of, int* tiles, int flags, atx_stream_t stream) {
     ATX_REQUIRE(logits && sel && wgt && seg_off && perm && slot_of && tiles, "atx_moe_route_plan: null pointer");
     ATX_REQUIRE((score == ATX_MOE_SOFTMAX || score == ATX_MOE_SIGMOID) && (power == 1 || power == 2),
                 "atx_moe_route_plan: score=%d power=%d", score, power);
@@ -548,7 +562,7 @@ int atx_moe_route_plan(const float* logits, long long ld, const float* correctio
     cfg.dynamicSmemBytes = sizeof(int) * (3 * static_cast<size_t>(E) + 1 + static_cast<size_t>(T) * top);
     cfg.stream = reinterpret_cast<cudaStream_t>(stream);
     set_pdl_moe(cfg, attr, flags);
-    const RouteArgs a{logits, ld, correction, R, top, scale, normalize, score, power};
+    const RouteArgs a{logits, ld, correction, R, top, scale, normalize, score, power, bias};
     ATX_CUDA(cudaLaunchKernelEx(&cfg, moe_route_plan_kernel, a, T, E, tile_rows, sel, wgt, seg_off, perm, slot_of, tiles));
     return ATX_OK;
 }

@@ -201,7 +201,7 @@ poly_norm_act_kernel(const float* __restrict__ z, long long ldz, const float* __
 
 // ---- residual update of a parallel layer ------------------------------------------------------------------------------------
 // Per row t (r = rows ? rows[t] : t):
-//   v = h[r] (or the embedding row, table_mode 2) + y_scale * (y[r] + sum_k wgt[r, k] experts[slot_of[r, k]])
+//   v = h[r] (or the embedding row, table_mode 2; its RMS norm times table_w, if given) + y_scale * (y[r] + sum_k wgt[r, k] experts[slot_of[r, k]])
 //       + embedding row (table_mode 1) + vec;         h[r] = v (not with rows)
 //   out_x[t] = v / sqrt(mean(v^2) + eps) * (w_shift + w_x)     x = a, b
 // Both norms share the row's statistic. CTAs beyond T clear zero_ptr. NV > 0: NV vectors of four elements per thread, the row
@@ -278,17 +278,35 @@ parallel_resid_norm_kernel(const __grid_constant__ ParallelResidArgs a) {
         er = reinterpret_cast<const XT*>(a.tm.table) + static_cast<long long>(id) * W;
     }
     const bool start = a.tm.table_mode == 2, enter = a.tm.table_mode == 1;
+    const XT* tw = start ? reinterpret_cast<const XT*>(a.tm.table_w) : nullptr;
+    float rs0 = 1.f;   // of the embedding row that the stream starts as
     const bool store = !a.rows && (yr || top || er || vec);
     const float sc = a.tm.y_scale;
     float ss = 0.f;
     if constexpr (NV > 0) {
         float4 v[NV];
+        if (tw) {
+            float s0 = 0.f;
+#pragma unroll
+            for (int n = 0; n < NV; ++n) {
+                const int i = threadIdx.x + n * blockDim.x;
+                if (i >= W4) continue;
+                const float4 e = rld4(er, i);
+                s0 += e.x * e.x + e.y * e.y + e.z * e.z + e.w * e.w;
+            }
+            rs0 = rsqrtf(row_sum(s0, red) / static_cast<float>(W) + a.eps);
+            __syncthreads();   // red is used again for the outgoing norm
+        }
 #pragma unroll
         for (int n = 0; n < NV; ++n) {
             const int i = threadIdx.x + n * blockDim.x;
             v[n] = make_float4(0.f, 0.f, 0.f, 0.f);
             if (i >= W4) continue;
             v[n] = start ? rld4(er, i) : rld4(hr, i);
+            if (tw) {
+                const float4 g = rld4(tw, i);
+                v[n].x *= rs0 * g.x, v[n].y *= rs0 * g.y, v[n].z *= rs0 * g.z, v[n].w *= rs0 * g.w;
+            }
             float4 add = make_float4(0.f, 0.f, 0.f, 0.f);
             if (yr) {
                 add = rld4(yr, i);
@@ -332,8 +350,18 @@ parallel_resid_norm_kernel(const __grid_constant__ ParallelResidArgs a) {
             }
         }
     } else {
+        if (tw) {
+            float s0 = 0.f;
+            for (int i = threadIdx.x; i < W; i += blockDim.x) {
+                const float e = rld(er, i);
+                s0 += e * e;
+            }
+            rs0 = rsqrtf(row_sum(s0, red) / static_cast<float>(W) + a.eps);
+            __syncthreads();
+        }
         for (int i = threadIdx.x; i < W; i += blockDim.x) {
             float v = start ? rld(er, i) : hr[i], add = 0.f;
+            if (tw) v *= rs0 * rld(tw, i);
             if (yr) {
                 add = yr[i];
                 if (a.tm.zero_y) yr[i] = 0.f;
@@ -437,7 +465,7 @@ int atx_parallel_resid_norm(float* h, const atx_resid_terms* terms, const void* 
     ParallelResidArgs a = {h, tm, w_a, out_a, w_b, out_b, w_shift, eps, rows, T, W, reinterpret_cast<uint4*>(zero_ptr), zero_bytes / 16};
     auto al16 = [](const void* p) { return reinterpret_cast<uintptr_t>(p) % 16 == 0; };
     const bool v4 = W % 4 == 0 && al16(h) && al16(tm.y) && al16(tm.experts) && (!tm.experts || tm.lde % 4 == 0) && al16(tm.table) &&
-                    al16(tm.vec) && al16(w_a) && al16(out_a) && al16(w_b) && al16(out_b);
+                    al16(tm.table_w) && al16(tm.vec) && al16(w_a) && al16(out_a) && al16(w_b) && al16(out_b);
     // few rows: as many threads per row as it has vectors; many rows: 256 threads and several vectors each
     const int W4 = W / 4;
     const int want = T <= 512 ? (W4 + 31) / 32 * 32 : 256;

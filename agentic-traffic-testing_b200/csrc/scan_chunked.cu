@@ -23,6 +23,8 @@
 // columns of the output: both compute their half of the sum over key dimensions for all 64 tokens and hand the partner
 // the 32 columns it owns through shared memory. Halving the per-warp tiles is what lets sixteen warps live on an SM;
 // with four warps of 246 registers the kernel ran at one warp per scheduler and waited on instruction latency.
+// ROT: the first rot_dims dimensions of q and k are rotated (element i with element i + rot_dims / 2, by the angles at the row's
+// position) in fp32 as they are read, ahead of their rounding to bf16; kmul, a constant on k, is part of c_t.
 // Sequences are walked as in seqmix.cu: rows [seq_start, seq_start + seq_count), state slot seq_slot, zero state when
 // seq_pos0 == 0.
 #include "common.cuh"
@@ -37,7 +39,7 @@ constexpr int kScT = 256;  // threads per CTA
 
 __device__ __forceinline__ float silu_sc(float x) { return x / (1.f + expf(-x)); }
 
-template <int D>
+template <int D, bool ROT>
 __global__ void __launch_bounds__(kScT, 2)
 scan_chunked_kernel(const float* __restrict__ q, long long ldq, const float* __restrict__ k, long long ldk,
                     const float* __restrict__ v, long long ldv, int H, int G, int V,
@@ -45,7 +47,8 @@ scan_chunked_kernel(const float* __restrict__ q, long long ldq, const float* __r
                     const float* __restrict__ kscale_tok, const float* __restrict__ skip, int act,
                     float* __restrict__ state, float* __restrict__ y, long long ldy,
                     const int* __restrict__ seq_start, const int* __restrict__ seq_count,
-                    const int* __restrict__ seq_pos0, const int* __restrict__ seq_slot, int vec) {
+                    const int* __restrict__ seq_pos0, const int* __restrict__ seq_slot, int vec,
+                    const float* __restrict__ rot, int rot_dims, float kmul) {
     constexpr int LQ = D + 8, LV = kScV + 8, LP = kScC + 8;   // padded rows: ldmatrix without bank conflicts
     extern __shared__ __align__(16) unsigned char smem_raw[];
     __nv_bfloat16* sQ = reinterpret_cast<__nv_bfloat16*>(smem_raw);   // [C][D]
@@ -72,7 +75,8 @@ scan_chunked_kernel(const float* __restrict__ q, long long ldq, const float* __r
 
     float S[DH / 8][4];
     float* st = state + (static_cast<long long>(seq_slot[s]) * H + h) * D * V;
-    const bool fresh = seq_pos0[s] == 0;
+    const int pos0 = seq_pos0[s];
+    const bool fresh = pos0 == 0;
 #pragma unroll
     for (int nd = 0; nd < DH / 8; ++nd)
 #pragma unroll
@@ -93,7 +97,7 @@ scan_chunked_kernel(const float* __restrict__ q, long long ldq, const float* __r
         if (threadIdx.x < kScC && c0n + static_cast<int>(threadIdx.x) < n) {
             const long long row = r0 + c0n + threadIdx.x;
             if (decay_tok) a_next = decay_tok[row * H + h];
-            c_next = kscale_tok ? kscale_tok[row * H + h] : 1.f;
+            c_next = kscale_tok ? kscale_tok[row * H + h] * kmul : kmul;
         }
     };
     auto pull_l2 = [&](int c0n) {
@@ -136,7 +140,65 @@ scan_chunked_kernel(const float* __restrict__ q, long long ldq, const float* __r
         const float Llast = Lc(kScC - 1);
         // Tiles: loads are issued in batches ahead of their use (a chunk is short, so memory latency is what a naive
         // element loop would spend its time on); 16-byte loads when pointers, pitches and sizes allow.
-        if (vec & 1) {
+        if (ROT && (vec & 4)) {
+            // an item is the eight elements of four rotated pairs (or eight elements past the rotated range)
+            constexpr int IT = kScC * D / 8 / kScT;
+            const int half = rot_dims / 2, n_pair = half / 4;
+            float4 q0[IT], q1[IT], k0[IT], k1[IT];
+#pragma unroll
+            for (int u = 0; u < IT; ++u) {
+                const int e = threadIdx.x + u * kScT, i = e / (D / 8), p = e - i * (D / 8);
+                const int d0 = p < n_pair ? 4 * p : rot_dims + 8 * (p - n_pair), d1 = p < n_pair ? d0 + half : d0 + 4;
+                q0[u] = q1[u] = k0[u] = k1[u] = make_float4(0.f, 0.f, 0.f, 0.f);
+                if (i < cn) {
+                    const float* qr = q + (r0 + c0 + i) * ldq + g * D;
+                    const float* kr = k + (r0 + c0 + i) * ldk + g * D;
+                    q0[u] = *reinterpret_cast<const float4*>(qr + d0), q1[u] = *reinterpret_cast<const float4*>(qr + d1);
+                    k0[u] = *reinterpret_cast<const float4*>(kr + d0), k1[u] = *reinterpret_cast<const float4*>(kr + d1);
+                }
+            }
+#pragma unroll
+            for (int u = 0; u < IT; ++u) {
+                const int e = threadIdx.x + u * kScT, i = e / (D / 8), p = e - i * (D / 8);
+                const int d0 = p < n_pair ? 4 * p : rot_dims + 8 * (p - n_pair), d1 = p < n_pair ? d0 + half : d0 + 4;
+                if (p < n_pair && i < cn) {
+                    const float* cs = rot + static_cast<long long>(pos0 + c0 + i) * rot_dims + 4 * p;
+                    const float4 c = __ldg(reinterpret_cast<const float4*>(cs)), sn = __ldg(reinterpret_cast<const float4*>(cs + half));
+                    auto turn = [&](float4& a, float4& b) {
+                        const float4 x = a, w = b;
+                        a = make_float4(fmaf(x.x, c.x, -(w.x * sn.x)), fmaf(x.y, c.y, -(w.y * sn.y)), fmaf(x.z, c.z, -(w.z * sn.z)),
+                                        fmaf(x.w, c.w, -(w.w * sn.w)));
+                        b = make_float4(fmaf(w.x, c.x, x.x * sn.x), fmaf(w.y, c.y, x.y * sn.y), fmaf(w.z, c.z, x.z * sn.z),
+                                        fmaf(w.w, c.w, x.w * sn.w));
+                    };
+                    turn(q0[u], q1[u]);
+                    turn(k0[u], k1[u]);
+                }
+                *reinterpret_cast<uint2*>(sQ + i * LQ + d0) = make_uint2(pack_bf16(q0[u].x, q0[u].y), pack_bf16(q0[u].z, q0[u].w));
+                *reinterpret_cast<uint2*>(sQ + i * LQ + d1) = make_uint2(pack_bf16(q1[u].x, q1[u].y), pack_bf16(q1[u].z, q1[u].w));
+                *reinterpret_cast<uint2*>(sK + i * LQ + d0) = make_uint2(pack_bf16(k0[u].x, k0[u].y), pack_bf16(k0[u].z, k0[u].w));
+                *reinterpret_cast<uint2*>(sK + i * LQ + d1) = make_uint2(pack_bf16(k1[u].x, k1[u].y), pack_bf16(k1[u].z, k1[u].w));
+            }
+        } else if (ROT) {   // any pitch, alignment and even rot_dims: an element and its partner at a time
+            const int half = rot_dims / 2;
+            for (int e = threadIdx.x; e < kScC * D; e += kScT) {
+                const int i = e / D, d = e - i * D;
+                float xq = 0.f, xk = 0.f;
+                if (i < cn) {
+                    const float* qr = q + (r0 + c0 + i) * ldq + g * D;
+                    const float* kr = k + (r0 + c0 + i) * ldk + g * D;
+                    xq = qr[d], xk = kr[d];
+                    if (d < rot_dims) {
+                        const int j = d < half ? d : d - half, dp = d < half ? d + half : d - half;
+                        const float* cs = rot + static_cast<long long>(pos0 + c0 + i) * rot_dims;
+                        const float c = cs[j], sn = d < half ? -cs[half + j] : cs[half + j];
+                        xq = fmaf(xq, c, qr[dp] * sn), xk = fmaf(xk, c, kr[dp] * sn);
+                    }
+                }
+                sQ[i * LQ + d] = __float2bfloat16_rn(xq);
+                sK[i * LQ + d] = __float2bfloat16_rn(xk);
+            }
+        } else if (vec & 1) {
             constexpr int IT = kScC * D / 4 / kScT, U = IT;   // at most 8: one batch
 #pragma unroll 1
             for (int it = 0; it < IT; it += U) {
@@ -394,17 +456,18 @@ scan_chunked_kernel(const float* __restrict__ q, long long ldq, const float* __r
         }
 }
 
-template <int D>
+template <int D, bool ROT>
 static int launch_scan_chunked(const float* q, long long ldq, const float* k, long long ldk, const float* v, long long ldv,
                                int H, int G, int V, const float* decay_head, const float* decay_tok,
                                const float* kscale_tok, const float* skip, int act, float* state, float* y,
                                long long ldy, const int* seq_start, const int* seq_count, const int* seq_pos0,
-                               const int* seq_slot, int n_seqs, int flags, cudaStream_t stream) {
+                               const int* seq_slot, int n_seqs, const float* rot, int rot_dims, float kmul, int flags,
+                               cudaStream_t stream) {
     const int smem = 2 * kScC * (D + 8) * 2 + 2 * kScC * (kScV + 8) * 2 + kScC * (kScC + 8) * 2 + 2 * kScC * 4 +
                      8 * 16 * 32 * 4;
     static bool attr_done = false;
     if (!attr_done) {
-        ATX_CUDA(cudaFuncSetAttribute(scan_chunked_kernel<D>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
+        ATX_CUDA(cudaFuncSetAttribute(scan_chunked_kernel<D, ROT>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
         attr_done = true;
     }
     cudaLaunchConfig_t cfg = {};
@@ -419,12 +482,13 @@ static int launch_scan_chunked(const float* q, long long ldq, const float* k, lo
         cfg.attrs = attr;
         cfg.numAttrs = 1;
     }
-    // bit 0: q / k rows can be read 16 bytes at a time; bit 1: v rows
+    // bit 0: q / k rows can be read 16 bytes at a time; bit 1: v rows; bit 2: rotated pairs as well
     auto al16 = [](const void* p) { return reinterpret_cast<uintptr_t>(p) % 16 == 0; };
     const int vec = ((al16(q) && al16(k) && ldq % 4 == 0 && ldk % 4 == 0) ? 1 : 0) |
-                    ((al16(v) && ldv % 4 == 0 && V % 4 == 0) ? 2 : 0);
-    ATX_CUDA(cudaLaunchKernelEx(&cfg, scan_chunked_kernel<D>, q, ldq, k, ldk, v, ldv, H, G, V, decay_head, decay_tok,
-                                kscale_tok, skip, act, state, y, ldy, seq_start, seq_count, seq_pos0, seq_slot, vec));
+                    ((al16(v) && ldv % 4 == 0 && V % 4 == 0) ? 2 : 0) |
+                    ((al16(q) && al16(k) && al16(rot) && ldq % 4 == 0 && ldk % 4 == 0 && rot_dims % 8 == 0) ? 4 : 0);
+    ATX_CUDA(cudaLaunchKernelEx(&cfg, scan_chunked_kernel<D, ROT>, q, ldq, k, ldk, v, ldv, H, G, V, decay_head, decay_tok,
+                                kscale_tok, skip, act, state, y, ldy, seq_start, seq_count, seq_pos0, seq_slot, vec, rot, rot_dims, kmul));
     return ATX_OK;
 }
 
@@ -443,6 +507,19 @@ int atx_linear_recurrence_chunked(const float* q, long long ldq, const float* k,
                                   const float* decay_tok, const float* kscale_tok, const float* skip, int act,
                                   float* state, float* y, long long ldy, const int* seq_start, const int* seq_count,
                                   const int* seq_pos0, const int* seq_slot, int n_seqs, int flags, atx_stream_t stream) {
+    return atx_linear_recurrence_rot_chunked(q, ldq, k, ldk, v, ldv, H, G, D, V, decay_head, decay_tok, kscale_tok, skip, act,
+                                             nullptr, 0, 1.f, state, y, ldy, seq_start, seq_count, seq_pos0, seq_slot, n_seqs, flags,
+                                             stream);
+}
+
+int atx_linear_recurrence_rot_chunked(const float* q, long long ldq, const float* k, long long ldk, const float* v,
+                                      long long ldv, int H, int G, int D, int V, const float* decay_head,
+                                      const float* decay_tok, const float* kscale_tok, const float* skip, int act,
+                                      const float* rot, int rot_dims, float kmul, float* state, float* y, long long ldy,
+                                      const int* seq_start, const int* seq_count, const int* seq_pos0, const int* seq_slot,
+                                      int n_seqs, int flags, atx_stream_t stream) {
+    ATX_REQUIRE(rot_dims >= 0 && rot_dims % 2 == 0 && rot_dims <= D && (rot_dims == 0 || (rot && !act)),
+                "atx_linear_recurrence_chunked: rotation of %d of %d dimensions needs an even count, a table and no act", rot_dims, D);
     ATX_REQUIRE(q && k && v && state && y && seq_start && seq_count && seq_pos0 && seq_slot,
                 "atx_linear_recurrence_chunked: null pointer");
     ATX_REQUIRE((decay_head != nullptr) != (decay_tok != nullptr),
@@ -450,10 +527,12 @@ int atx_linear_recurrence_chunked(const float* q, long long ldq, const float* k,
     ATX_REQUIRE(n_seqs > 0 && H > 0 && G > 0 && H % G == 0 && V > 0 && atx_linear_recurrence_chunked_supported(D),
                 "atx_linear_recurrence_chunked: bad shape n_seqs=%d H=%d G=%d D=%d V=%d", n_seqs, H, G, D, V);
     cudaStream_t cs = reinterpret_cast<cudaStream_t>(stream);
-#define ATX_SCAN_CASE(D_)                                                                                                \
-    case D_:                                                                                                             \
-        return launch_scan_chunked<D_>(q, ldq, k, ldk, v, ldv, H, G, V, decay_head, decay_tok, kscale_tok, skip, act,   \
-                                       state, y, ldy, seq_start, seq_count, seq_pos0, seq_slot, n_seqs, flags, cs)
+#define ATX_SCAN_RUN(D_, ROT_)                                                                                           \
+    launch_scan_chunked<D_, ROT_>(q, ldq, k, ldk, v, ldv, H, G, V, decay_head, decay_tok, kscale_tok, skip, act, state, \
+                                  y, ldy, seq_start, seq_count, seq_pos0, seq_slot, n_seqs, rot, rot_dims, kmul, flags, cs)
+#define ATX_SCAN_CASE(D_) \
+    case D_:              \
+        return rot_dims > 0 ? ATX_SCAN_RUN(D_, true) : ATX_SCAN_RUN(D_, false)
     switch (D) {
         ATX_SCAN_CASE(32);
         ATX_SCAN_CASE(64);
@@ -461,6 +540,7 @@ int atx_linear_recurrence_chunked(const float* q, long long ldq, const float* k,
         ATX_SCAN_CASE(128);
     }
 #undef ATX_SCAN_CASE
+#undef ATX_SCAN_RUN
     return ATX_OK;
 }
 

@@ -263,7 +263,7 @@ resid_norm_kernel(float* __restrict__ h, float* __restrict__ y, const XT* __rest
 // ---- act(gate) * up --------------------------------------------------------------------------------------------------
 template <typename XT>
 __global__ void __launch_bounds__(256) gated_act_kernel(const float* __restrict__ gu, XT* __restrict__ out, long long total,
-                                                        int I) {
+                                                        int I, int gelu) {
     pdl_launch_dependents();
     pdl_wait();
     for (long long e = static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x; e < total;
@@ -271,7 +271,9 @@ __global__ void __launch_bounds__(256) gated_act_kernel(const float* __restrict_
         const long long t = e / I;
         const int i = static_cast<int>(e - t * I);
         const float g = gu[t * 2 * I + i], u = gu[t * 2 * I + I + i];
-        stf(out, e, silu_f(g) * u);
+        // gelu: its tanh form, with (1 + tanh x) / 2 = 1 / (1 + exp(-2 x))
+        const float a = gelu ? g * sigmoid_f(1.5957691216057308f * (g + 0.044715f * g * g * g)) : silu_f(g);
+        stf(out, e, a * u);
     }
 }
 
@@ -297,7 +299,7 @@ __global__ void __launch_bounds__(256) gated_act_clamped_kernel(const float* __r
 // mode 1: u = y * silu(g); out = rms(u) * w * scale  (gate before the norm)
 // mode 2: out = rms(y) * w * silu(g) * scale         (silu gate after the norm)
 // The norm runs over n / groups consecutive elements; grid (T, groups). w_shared: one weight vector of n / groups
-// elements for every group instead of n weights.
+// elements for every group instead of n weights. w == nullptr: no weights.
 template <typename XT, bool VEC>
 __global__ void __launch_bounds__(1024)
 gated_norm_kernel(const float* __restrict__ y, long long ldy, const float* __restrict__ gate, long long ldg,
@@ -311,7 +313,7 @@ gated_norm_kernel(const float* __restrict__ y, long long ldy, const float* __res
     const int c0 = blockIdx.y * n_group;
     const float* yr = y + t * ldy + c0;
     const float* gr = gate + t * ldg + c0;
-    if (!w_shared) w += c0;
+    if (w && !w_shared) w += c0;
     if (VEC) {   // sizes and pitches multiples of 4, pointers 16-byte aligned: four elements per access, one gate pass
         const int n4 = n_group / 4;
         float4* s4 = reinterpret_cast<float4*>(sgn);
@@ -329,7 +331,7 @@ gated_norm_kernel(const float* __restrict__ y, long long ldy, const float* __res
         XT* o = out + t * ldo + c0;
         for (int i = threadIdx.x; i < n4; i += blockDim.x) {
             float4 v = s4[i];
-            const float4 ww = ld4(w, i);
+            const float4 ww = w ? ld4(w, i) : make_float4(1.f, 1.f, 1.f, 1.f);
             v.x *= rs * ww.x, v.y *= rs * ww.y, v.z *= rs * ww.z, v.w *= rs * ww.w;
             if (mode == 0) {
                 const float4 g = ld4(gr, i);
@@ -353,9 +355,9 @@ gated_norm_kernel(const float* __restrict__ y, long long ldy, const float* __res
     for (int i = threadIdx.x; i < n_group; i += blockDim.x) {
         float v = yr[i];
         if (mode == 1)
-            v = v * silu_f(gr[i]) * rs * ldf(w, i);
+            v = v * silu_f(gr[i]) * rs * (w ? ldf(w, i) : 1.f);
         else
-            v = v * rs * ldf(w, i) * (mode == 2 ? silu_f(gr[i]) : sigmoid_f(gr[i]));
+            v = v * rs * (w ? ldf(w, i) : 1.f) * (mode == 2 ? silu_f(gr[i]) : sigmoid_f(gr[i]));
         stf(o, i, v * scale);
     }
 }
@@ -383,7 +385,7 @@ gated_norm_warp_kernel(const float* __restrict__ y, long long ldy, const float* 
         }
         const float rs = rsqrtf(warp_sum(v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w) / static_cast<float>(n_group) + eps) * scale;
         if (!on) continue;
-        const float4 ww = ld4(w_shared ? w : w + c0, lane);
+        const float4 ww = w ? ld4(w_shared ? w : w + c0, lane) : make_float4(1.f, 1.f, 1.f, 1.f);
         v.x *= rs * ww.x, v.y *= rs * ww.y, v.z *= rs * ww.z, v.w *= rs * ww.w;
         if (mode == 0)
             v.x *= sigmoid_f(g.x), v.y *= sigmoid_f(g.y), v.z *= sigmoid_f(g.z), v.w *= sigmoid_f(g.w);
@@ -755,6 +757,8 @@ __device__ __forceinline__ f32x2 mul2(f32x2 a, f32x2 b) {
 //   act = 1 applies silu to q, k and v as they are read.
 //   CH: the decay acts per key channel instead, a_t[d] = exp(ldecay_chan[t, h D + d]) (logarithms given, pitch ldc), and q
 //   is multiplied by qscale as it is read.
+//   rot (nullable, [max_pos, rot_dims] cosines then sines): the first rot_dims dimensions of q and k are rotated as they are read,
+//   element i with element i + rot_dims / 2, by the angles at the row's position; kmul multiplies k.
 // One CTA owns a V-tile of one head of one sequence and walks the sequence's rows in order. A thread keeps DS rows of
 // one column of S in registers for the whole walk (the state is read once and written once per step); rows are staged
 // through shared memory kChunk at a time, and the partial dot products of the D-slices are summed per chunk.
@@ -769,7 +773,8 @@ linear_recurrence_kernel(const float* __restrict__ q, long long ldq, const float
                          float* __restrict__ state, float* __restrict__ y, long long ldy,
                          const int* __restrict__ seq_start, const int* __restrict__ seq_count,
                          const int* __restrict__ seq_pos0, const int* __restrict__ seq_slot, int VT, int DG,
-                         const float* __restrict__ ldecay_chan = nullptr, long long ldc = 0, float qscale = 1.f) {
+                         const float* __restrict__ ldecay_chan = nullptr, long long ldc = 0, float qscale = 1.f,
+                         const float* __restrict__ rot = nullptr, int rot_dims = 0, float kmul = 1.f) {
     extern __shared__ __align__(16) float sm[];
     pdl_launch_dependents();
     pdl_wait();
@@ -790,7 +795,8 @@ linear_recurrence_kernel(const float* __restrict__ q, long long ldq, const float
     float* sd = sp + kRecChunk * DG * VT;      // CH: [kRecChunk][D] decay factors per key channel
     float S[DS];
     float* st = state + ((static_cast<long long>(seq_slot[s]) * H + h) * D) * V;
-    const bool fresh = seq_pos0[s] == 0;
+    const int pos0 = seq_pos0[s];
+    const bool fresh = pos0 == 0;
 #pragma unroll
     for (int i = 0; i < DS; ++i) S[i] = (live && !fresh && d0 + i < D) ? st[static_cast<long long>(d0 + i) * V + col] : 0.f;
     const float dskip = skip ? skip[h] : 0.f;
@@ -806,6 +812,14 @@ linear_recurrence_kernel(const float* __restrict__ q, long long ldq, const float
                 kv = silu_f(kv);
             }
             if (kscale_tok) kv *= kscale_tok[row * H + h];
+            if (d < rot_dims) {
+                const int half = rot_dims / 2, j = d < half ? d : d - half, dp = d < half ? d + half : d - half;
+                const float* cs = rot + static_cast<long long>(pos0 + c0 + i) * rot_dims;
+                const float c = cs[j], sn = d < half ? -cs[half + j] : cs[half + j];
+                qv = fmaf(qv, c, q[row * ldq + g * D + dp] * sn);
+                kv = fmaf(kv, c, k[row * ldk + g * D + dp] * sn);
+            }
+            kv *= kmul;
             if (CH) {
                 qv *= qscale;
                 sd[i * D + d] = expf(ldecay_chan[row * ldc + static_cast<long long>(h) * D + d]);
@@ -1005,7 +1019,12 @@ int atx_resid_norm_out(float* h, float* y, const void* w_post, const void* post_
 }
 
 int atx_gated_act(const float* gu, void* out, int T, int I, int dtype, int flags, atx_stream_t stream) {
+    return atx_gated_act_kind(gu, out, T, I, ATX_ACT_SILU, dtype, flags, stream);
+}
+
+int atx_gated_act_kind(const float* gu, void* out, int T, int I, int kind, int dtype, int flags, atx_stream_t stream) {
     ATX_REQUIRE(gu && out, "atx_gated_act: null pointer");
+    ATX_REQUIRE(kind == ATX_ACT_SILU || kind == ATX_ACT_GELU_TANH, "atx_gated_act: unknown activation %d", kind);
     ATX_REQUIRE(T > 0 && I > 0, "atx_gated_act: bad shape T=%d I=%d", T, I);
     const long long total = static_cast<long long>(T) * I;
     long long blocks = (total + 255) / 256;
@@ -1017,7 +1036,8 @@ int atx_gated_act(const float* gu, void* out, int T, int I, int dtype, int flags
     cfg.blockDim = dim3(256);
     cfg.stream = reinterpret_cast<cudaStream_t>(stream);
     set_pdl2(cfg, attr, flags);
-    ATX_DISPATCH_XT(dtype, ATX_CUDA(cudaLaunchKernelEx(&cfg, gated_act_kernel<XT>, gu, reinterpret_cast<XT*>(out), total, I)));
+    ATX_DISPATCH_XT(dtype, ATX_CUDA(cudaLaunchKernelEx(&cfg, gated_act_kernel<XT>, gu, reinterpret_cast<XT*>(out), total, I,
+                                                       kind == ATX_ACT_GELU_TANH ? 1 : 0)));
     return ATX_OK;
 }
 
@@ -1049,7 +1069,7 @@ int atx_gated_norm(const float* y, long long ldy, const float* gate, long long l
 int atx_gated_norm_groups(const float* y, long long ldy, const float* gate, long long ldg, const void* w, int w_shared,
                           void* out, long long ldo, int T, int n, int groups, float eps, int mode, float scale, int dtype,
                           int flags, atx_stream_t stream) {
-    ATX_REQUIRE(y && gate && w && out, "atx_gated_norm: null pointer");
+    ATX_REQUIRE(y && gate && out, "atx_gated_norm: null pointer");
     ATX_REQUIRE(T > 0 && n > 0 && groups > 0 && n % groups == 0 && mode >= 0 && mode <= 2,
                 "atx_gated_norm: bad arguments T=%d n=%d groups=%d mode=%d", T, n, groups, mode);
     cudaLaunchConfig_t cfg = {};
@@ -1162,8 +1182,20 @@ int atx_linear_recurrence(const float* q, long long ldq, const float* k, long lo
                           const float* kscale_tok, const float* skip, int act, float* state, float* y, long long ldy,
                           const int* seq_start, const int* seq_count, const int* seq_pos0, const int* seq_slot,
                           int n_seqs, int flags, atx_stream_t stream) {
+    return atx_linear_recurrence_rot(q, ldq, k, ldk, v, ldv, H, G, D, V, decay_head, decay_tok, kscale_tok, skip, act, nullptr, 0,
+                                     1.f, state, y, ldy, seq_start, seq_count, seq_pos0, seq_slot, n_seqs, flags, stream);
+}
+
+int atx_linear_recurrence_rot(const float* q, long long ldq, const float* k, long long ldk, const float* v, long long ldv,
+                              int H, int G, int D, int V, const float* decay_head, const float* decay_tok,
+                              const float* kscale_tok, const float* skip, int act, const float* rot, int rot_dims, float kmul,
+                              float* state, float* y, long long ldy, const int* seq_start, const int* seq_count,
+                              const int* seq_pos0, const int* seq_slot, int n_seqs, int flags, atx_stream_t stream) {
     ATX_REQUIRE(q && k && v && state && y && seq_start && seq_count && seq_pos0 && seq_slot,
                 "atx_linear_recurrence: null pointer");
+    ATX_REQUIRE(rot_dims >= 0 && rot_dims % 2 == 0 && rot_dims <= D && (rot_dims == 0 || (rot && !act && !kscale_tok)),
+                "atx_linear_recurrence: rotation of %d of %d dimensions needs an even count, a table, and neither act nor kscale_tok",
+                rot_dims, D);
     ATX_REQUIRE((decay_head != nullptr) != (decay_tok != nullptr),
                 "atx_linear_recurrence: exactly one of decay_head / decay_tok");
     ATX_REQUIRE(n_seqs > 0 && H > 0 && G > 0 && H % G == 0 && D > 0 && V > 0 && D <= 512,
@@ -1192,7 +1224,8 @@ int atx_linear_recurrence(const float* q, long long ldq, const float* k, long lo
                                           cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)));          \
         ATX_CUDA(cudaLaunchKernelEx(&cfg, linear_recurrence_kernel<DS_, FULL_>, q, ldq, k, ldk, v, ldv, H, G, D, V,       \
                                     decay_head, decay_tok, kscale_tok, skip, act, state, y, ldy, seq_start, seq_count,   \
-                                    seq_pos0, seq_slot, VT, DG, static_cast<const float*>(nullptr), 0LL, 1.f)); \
+                                    seq_pos0, seq_slot, VT, DG, static_cast<const float*>(nullptr), 0LL, 1.f, rot,     \
+                                    rot_dims, kmul));                                                                     \
     } while (0)
     if (DS == 32 && full)
         ATX_REC_LAUNCH(32, true);
@@ -1300,7 +1333,7 @@ int atx_gated_linear_recurrence(const float* q, long long ldq, const float* k, l
                                           cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)));          \
         ATX_CUDA(cudaLaunchKernelEx(&cfg, linear_recurrence_kernel<DS_, FULL_, true>, q, ldq, k, ldk, v, ldv, H, H, D, V, \
                                     none, none, none, none, 0, state, y, ldy, seq_start, seq_count, seq_pos0, seq_slot,  \
-                                    VT, DG, ldecay, ldc, qscale));                                                        \
+                                    VT, DG, ldecay, ldc, qscale, none, 0, 1.f));                                          \
     } while (0)
     if (DS == 32 && full)
         ATX_GREC_LAUNCH(32, true);

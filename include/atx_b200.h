@@ -68,6 +68,9 @@ typedef struct atx_gemm_plan atx_gemm_plan;
 #define ATX_GEMM_GLU_CLAMP_BF16 5
 /* out fp32 = limit tanh(acc / limit), limit from atx_gemm_plan_set_gate: the cap on a model's logits. No split-K. */
 #define ATX_GEMM_SOFTCAP_F32 6
+/* ATX_GEMM_SWIGLU_BF16 with the tanh form of gelu on the gate (same row layout, same split-K): out = gelu(acc_gate) acc_up,
+ * gelu(z) = z/2 (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3))). */
+#define ATX_GEMM_GEGLU_BF16 7
 int atx_gemm_plan_create(atx_gemm_plan** plan, const void* W, long long N, long long K, const void* X,
                          long long T_cap, long long ldx);
 void atx_gemm_plan_destroy(atx_gemm_plan* plan);
@@ -255,7 +258,7 @@ int atx_resid_norm(float* h, float* y, const void* w_post, const void* vec, cons
                    int flags, atx_stream_t stream);
 /* out[t, i] = silu(gu[t, i]) * gu[t, I + i] */
 int atx_gated_act(const float* gu, void* out, int T, int I, int dtype, int flags, atx_stream_t stream);
-/* Gated RMS norm over n / groups consecutive elements at a time:
+/* Gated RMS norm over n / groups consecutive elements at a time (w nullable: no weights):
  *   mode 0: out = rms(y) * w * sigmoid(gate) * scale;   mode 1: out = rms(y * silu(gate)) * w * scale */
 int atx_gated_norm(const float* y, long long ldy, const float* gate, long long ldg, const void* w, void* out,
                    long long ldo, int T, int n, int groups, float eps, int mode, float scale, int dtype, int flags,
@@ -330,6 +333,7 @@ int atx_tanh_norm(const float* x, const int* rows, float alpha, const void* w, c
                   void* zero_ptr, long long zero_bytes, int dtype, int flags, atx_stream_t stream);
 #define ATX_ACT_RELU2 0     /* max(z, 0)^2 */
 #define ATX_ACT_GELU_TANH 1 /* z/2 (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3))) */
+#define ATX_ACT_SILU 2      /* z / (1 + exp(-z)) (gated activations) */
 /* out[t, i] = act(in[t, i]) (fp32 in, element type out). */
 int atx_unary_act(const float* in, long long ldi, void* out, long long ldo, int T, int I, int kind, int dtype, int flags,
                   atx_stream_t stream);
@@ -550,7 +554,7 @@ int atx_moe_route_opts(const float* logits, long long ld, const float* correctio
 /* What a parallel layer adds to the stream (see atx_parallel_resid_norm). y (nullable): the dense sublayers' output [T, W];
  * zero_y != 0 clears each row once read. experts (nullable): expert outputs by slot (row pitch lde), slot_of / wgt [T, top] as
  * atx_moe_plan / atx_moe_route* write them (slot -1: no contribution). table_mode 1: the embedding row of ids[r] is added;
- * 2: the stream starts as that row (h is not read). vec (nullable, element type [W]) is added last. */
+ * 2: the stream starts as that row, or with table_w (nullable, element type [W]) as rms(row) * table_w (h is not read). vec (nullable, element type [W]) is added last. */
 typedef struct atx_resid_terms {
     float* y;
     const float* experts;
@@ -562,6 +566,7 @@ typedef struct atx_resid_terms {
     long long lde;
     float y_scale;
     int zero_y, top, vocab, table_mode;
+    const void* table_w;
 } atx_resid_terms;
 /* v = h[r] + y_scale (y[r] + sum_k wgt[r, k] experts[slot_of[r, k]]) (+ table[ids[r]]) (+ vec), r = rows ? rows[t] : t; h[r] = v
  * (without rows); out_a[t] = rms(v) (w_shift + w_a), out_b[t] = rms(v) (w_shift + w_b) (each nullable; one row statistic for
@@ -611,11 +616,47 @@ int atx_moe_route_plan(const float* logits, long long ld, const float* correctio
 /* atx_gemm_run_grouped for steps of at most 64 tokens, on the weight-streaming kernel: one tile per chosen group (a plan made with
  * tile_rows >= 64), n_group rows of W each. perm == NULL: X holds the groups' rows back to back (row = slot). perm != NULL: X
  * holds the step's T tokens as they are (no gather); out[slot, :] = X[perm[slot] / top, :] W_e^T for the slots of every group. K
- * is split over a cluster where one wave has room. Modes STORE_F32, STORE_BF16, RELU2_BF16. */
+ * is split over a cluster where one wave has room. Modes STORE_F32, STORE_BF16, RELU2_BF16, and the gated ones (out has n_group / 2
+ * columns; n_group a multiple of 128). */
 int atx_gemm_run_grouped_small(const atx_gemm_plan* plan, void* out, long long ldo, int n_group, int mode, const int* seg_off,
                                const int* tiles, int max_tiles, const int* perm, int top, int T, int flags, atx_stream_t stream);
 /* x[t, n] = cap tanh(x[t, n] / cap) in place, n < N. */
 int atx_soft_cap(float* x, long long ld, int T, int N, float cap, int flags, atx_stream_t stream);
+
+/* ---- Further mechanisms: a query factor that grows with the position, a recurrence that rotates its queries and keys, a bias on
+ * router outputs, gelu gates. (Sutosun is built from these; every constant is an argument.) */
+
+/* atx_qk_prepare with the prepared query at position p multiplied by 1 + qt_coef ln(floor((p + 1) / qt_every) + 1) (qt_coef 0: no
+ * factor; qt_every > 0). */
+int atx_qk_prepare_temp(const float* proj, long long ld, int q_off, int k_off, int v_off, const void* bq, const void* bk,
+                        const void* bv, const void* wq, const void* wk, const float* rot, int rot_dims, float qt_coef,
+                        float qt_every, const int* positions, const int* slots, void* q_out, void* k_cache, void* v_cache,
+                        int T, int H, int G, int D, int Vd, int block_size, float eps, int dtype, int flags,
+                        atx_stream_t stream);
+/* atx_linear_recurrence[_chunked] whose q and k are rotated in fp32 as they are read: of the first rot_dims dimensions of a head,
+ * element i and element i + rot_dims / 2 turn by the angles of rot [max_pos, rot_dims] (cosines, then sines) at the row's position;
+ * k is multiplied by kmul afterwards. rot_dims 0: no rotation. With rotation: no act, and no kscale_tok in the first form. */
+int atx_linear_recurrence_rot(const float* q, long long ldq, const float* k, long long ldk, const float* v, long long ldv,
+                              int H, int G, int D, int V, const float* decay_head, const float* decay_tok,
+                              const float* kscale_tok, const float* skip, int act, const float* rot, int rot_dims, float kmul,
+                              float* state, float* y, long long ldy, const int* seq_start, const int* seq_count,
+                              const int* seq_pos0, const int* seq_slot, int n_seqs, int flags, atx_stream_t stream);
+int atx_linear_recurrence_rot_chunked(const float* q, long long ldq, const float* k, long long ldk, const float* v,
+                                      long long ldv, int H, int G, int D, int V, const float* decay_head,
+                                      const float* decay_tok, const float* kscale_tok, const float* skip, int act,
+                                      const float* rot, int rot_dims, float kmul, float* state, float* y, long long ldy,
+                                      const int* seq_start, const int* seq_count, const int* seq_pos0, const int* seq_slot,
+                                      int n_seqs, int flags, atx_stream_t stream);
+/* atx_gated_act with a choice of activation: out[t, i] = act(gu[t, i]) * gu[t, I + i], ATX_ACT_SILU or ATX_ACT_GELU_TANH. */
+int atx_gated_act_kind(const float* gu, void* out, int T, int I, int kind, int dtype, int flags, atx_stream_t stream);
+/* atx_moe_route_scored / atx_moe_route_plan with bias [R] (nullable) added to the logits. The soft-max over the chosen outputs alone
+ * is the soft-max over all with normalize != 0. */
+int atx_moe_route_biased(const float* logits, long long ld, const float* bias, const float* correction, int R, int top,
+                         float scale, int normalize, int score, int power, int* sel, float* wgt, int T, int flags,
+                         atx_stream_t stream);
+int atx_moe_route_plan_biased(const float* logits, long long ld, const float* bias, const float* correction, int R, int top,
+                              float scale, int normalize, int score, int power, int T, int E, int tile_rows, int* sel,
+                              float* wgt, int* seg_off, int* perm, int* slot_of, int* tiles, int flags, atx_stream_t stream);
 
 #ifdef __cplusplus
 }

@@ -808,7 +808,7 @@ def test_sigmoid_routing_keeps_scores_and_orders_saturated_ones_by_their_logits(
 def test_squared_relu_experts_decode_tiles_and_the_grouped_gemm(T):
     """The helper the program uses, both dtypes, both tile sizes and the tcgen05 path: by-slot outputs, summed with squared scores,
     against the definition (the weight on the expert's input)."""
-    from atx.models.common import UngatedExperts
+    from atx.models.common import Experts
 
     L, Cb = lib()
     for E, top, F, W in ((5, 2, 64, 128), (3, 3, 192, 64), (9, 1, 40, 72), (160, 2, 320, 64), (2, 1, 512, 1024)):
@@ -823,7 +823,7 @@ def test_squared_relu_experts_decode_tiles_and_the_grouped_gemm(T):
             xt, dt = types(dtype)
             xn = torch.zeros(max(T, 16), W, dtype=xt, device=DEV)
             xn[:T] = x.to(xt)
-            ex = UngatedExperts(L, ck, [{"router": {"top": top, "experts": E}, "expert": {"ff": F}}], max(T, 16), W, xn, dt)
+            ex = Experts(L, ck, [{"router": {"top": top, "experts": E}, "expert": {"ff": F}}], max(T, 16), W, xn, dt, power=2)
             up = torch.stack([wt[f"e{e}.up"] for e in range(E)]).to(device=DEV, dtype=xt).contiguous()
             down = torch.stack([wt[f"e{e}.down"] for e in range(E)]).to(device=DEV, dtype=xt).contiguous()
             n = ex.run(logits.data_ptr(), E, top, up, down, ex.plans(up, down), T, T <= 64, 0, stream())
