@@ -171,6 +171,110 @@ qk_prepare_kernel(const float* __restrict__ proj, long long ld, int q_off, int k
     }
 }
 
+// The same for sizes, pitches and pointers that allow four elements per access (heads of 4 j elements): a thread keeps NV vectors of
+// the row in registers between the sums and the store, biases and norm weights arrive with the row.
+__device__ __forceinline__ float4 ldx4(const float* p, long long i4) { return reinterpret_cast<const float4*>(p)[i4]; }
+__device__ __forceinline__ float4 ldx4(const __nv_bfloat16* p, long long i4) {
+    const uint2 u = reinterpret_cast<const uint2*>(p)[i4];
+    return make_float4(bf16lo(u.x), bf16hi(u.x), bf16lo(u.y), bf16hi(u.y));
+}
+__device__ __forceinline__ void stx4(float* p, long long i4, float4 v) { reinterpret_cast<float4*>(p)[i4] = v; }
+__device__ __forceinline__ void stx4(__nv_bfloat16* p, long long i4, float4 v) {
+    reinterpret_cast<uint2*>(p)[i4] = make_uint2(pack_bf16(v.x, v.y), pack_bf16(v.z, v.w));
+}
+
+template <typename XT, int NV>
+__global__ void __launch_bounds__(1024)
+qk_prepare_vec_kernel(const float* __restrict__ proj, long long ld, int q_off, int k_off, int v_off, const XT* __restrict__ bq,
+                      const XT* __restrict__ bk, const XT* __restrict__ bv, const XT* __restrict__ wq, const XT* __restrict__ wk,
+                      const float* __restrict__ rot, int rot_dims, const int* __restrict__ positions,
+                      const int* __restrict__ slots, XT* __restrict__ q_out, XT* __restrict__ k_cache,
+                      XT* __restrict__ v_cache, int H, int G, int D, int Vd, int bs, float eps, float qt_coef, float qt_every) {
+    __shared__ float red[2][32];
+    pdl_launch_dependents();
+    pdl_wait();
+    const long long t = blockIdx.x;
+    const int slot = slots[t];
+    if (slot < 0) return;   // padded row
+    const int pos = positions[t];
+    const int nq4 = H * D / 4, n4 = nq4 + G * D / 4, nv4 = G * Vd / 4;
+    const float* row = proj + t * ld;
+    float4 v[NV];
+#pragma unroll
+    for (int n = 0; n < NV; ++n) {
+        const int i = threadIdx.x + n * blockDim.x;
+        v[n] = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (i < n4) v[n] = i < nq4 ? ldx4(row + q_off, i) : ldx4(row + k_off, i - nq4);
+    }
+    const int blk = slot / bs, off = slot - blk * bs;
+    for (int i = threadIdx.x; i < nv4; i += blockDim.x) {
+        float4 x = ldx4(row + v_off, i);
+        if (bv) {
+            const float4 b = ldx4(bv, i);
+            x.x += b.x, x.y += b.y, x.z += b.z, x.w += b.w;
+        }
+        const int head = 4 * i / Vd, d = 4 * i - head * Vd;
+        stx4(v_cache + ((static_cast<long long>(blk) * G + head) * bs + off) * Vd + d, 0, x);
+    }
+    float ssq = 0.f, ssk = 0.f;
+#pragma unroll
+    for (int n = 0; n < NV; ++n) {
+        const int i = threadIdx.x + n * blockDim.x;
+        const bool isq = i < nq4;
+        const XT* b = isq ? bq : bk;
+        if (b && i < n4) {
+            const float4 c = ldx4(b, isq ? i : i - nq4);
+            v[n].x += c.x, v[n].y += c.y, v[n].z += c.z, v[n].w += c.w;
+        }
+        const float ss = v[n].x * v[n].x + v[n].y * v[n].y + v[n].z * v[n].z + v[n].w * v[n].w;
+        ssq += isq ? ss : 0.f;
+        ssk += isq ? 0.f : ss;
+    }
+    ssq = warp_sum(ssq);
+    ssk = warp_sum(ssk);
+    if ((threadIdx.x & 31) == 0) red[0][threadIdx.x >> 5] = ssq, red[1][threadIdx.x >> 5] = ssk;
+    __syncthreads();
+    float tq = 0.f, tk = 0.f;
+    const int lane = threadIdx.x & 31;
+    if (lane < static_cast<int>(blockDim.x >> 5)) tq = red[0][lane], tk = red[1][lane];
+    tq = warp_sum(tq);
+    tk = warp_sum(tk);
+    float rq = wq ? rsqrtf(tq / static_cast<float>(4 * nq4) + eps) : 1.f;
+    const float rk = wk ? rsqrtf(tk / static_cast<float>(4 * (n4 - nq4)) + eps) : 1.f;
+    if (qt_coef != 0.f) rq *= fmaf(qt_coef, logf(floorf(static_cast<float>(pos + 1) / qt_every) + 1.f), 1.f);
+    const float* cs = rot + static_cast<long long>(pos) * rot_dims;
+    const int half = rot_dims / 2;
+#pragma unroll
+    for (int n = 0; n < NV; ++n) {
+        const int i = threadIdx.x + n * blockDim.x;
+        if (i >= n4) continue;
+        const bool isq = i < nq4;
+        const int j = isq ? i : i - nq4;
+        const XT* w = isq ? wq : wk;
+        const float r = isq ? rq : rk;
+        float4 x = make_float4(v[n].x * r, v[n].y * r, v[n].z * r, v[n].w * r);
+        if (w) {
+            const float4 g = ldx4(w, j);
+            x.x *= g.x, x.y *= g.y, x.z *= g.z, x.w *= g.w;
+        }
+        const int head = 4 * j / D, d = 4 * j - head * D;
+        if (d < rot_dims) {
+            const float c = cs[d / 2], sn = cs[half + d / 2];
+            const float a = x.x * c - x.y * sn, b = x.y * c + x.x * sn;
+            x.x = a, x.y = b;
+        }
+        if (d + 2 < rot_dims) {
+            const float c = cs[d / 2 + 1], sn = cs[half + d / 2 + 1];
+            const float a = x.z * c - x.w * sn, b = x.w * c + x.z * sn;
+            x.z = a, x.w = b;
+        }
+        if (isq)
+            stx4(q_out + t * 4 * nq4, j, x);
+        else
+            stx4(k_cache + ((static_cast<long long>(blk) * G + head) * bs + off) * D + d, 0, x);
+    }
+}
+
 // ---- attention ---------------------------------------------------------------------------------------------------
 constexpr int kMaxVdPerLane = 16;  // Vd <= 512; the kernel is instantiated for 2, 4, 8 and 16 value elements per lane
 
@@ -773,6 +877,40 @@ int atx_qk_prepare_temp(const float* proj, long long ld, int q_off, int k_off, i
         attr[0].val.programmaticStreamSerializationAllowed = 1;
         cfg.attrs = attr;
         cfg.numAttrs = 1;
+    }
+    auto al16 = [](const void* p) { return reinterpret_cast<uintptr_t>(p) % 16 == 0; };
+    const int n4 = (H + G) * D / 4;
+    if (D % 4 == 0 && Vd % 4 == 0 && ((q_off | k_off | v_off) & 3) == 0 && ld % 4 == 0 && n4 <= 4096 && al16(proj) && al16(bq) &&
+        al16(bk) && al16(bv) && al16(wq) && al16(wk) && al16(q_out) && al16(k_cache) && al16(v_cache)) {
+        // few rows: as many threads as the row has vectors; many rows: up to four vectors per thread, more CTAs per SM
+        int threads = T <= 512 ? (n4 + 31) / 32 * 32 : ((n4 + 3) / 4 + 31) / 32 * 32;
+        threads = threads > 1024 ? 1024 : (threads < 64 ? 64 : threads);
+        const int nv = (n4 + threads - 1) / threads;
+        cfg.blockDim = dim3(threads);
+        cfg.dynamicSmemBytes = 0;
+#define ATX_QK_VEC(XT_, NV_)                                                                                                   \
+    ATX_CUDA(cudaLaunchKernelEx(&cfg, qk_prepare_vec_kernel<XT_, NV_>, proj, ld, q_off, k_off, v_off,                          \
+                                reinterpret_cast<const XT_*>(bq), reinterpret_cast<const XT_*>(bk),                            \
+                                reinterpret_cast<const XT_*>(bv), reinterpret_cast<const XT_*>(wq),                            \
+                                reinterpret_cast<const XT_*>(wk), rot, rot_dims, positions, slots,                             \
+                                reinterpret_cast<XT_*>(q_out), reinterpret_cast<XT_*>(k_cache),                                \
+                                reinterpret_cast<XT_*>(v_cache), H, G, D, Vd, block_size, eps, qt_coef, qt_every))
+#define ATX_QK_VEC_XT(NV_)                                                  \
+    do {                                                                    \
+        if (dtype == ATX_DT_F32)                                            \
+            ATX_QK_VEC(float, NV_);                                         \
+        else                                                                \
+            ATX_QK_VEC(__nv_bfloat16, NV_);                                 \
+    } while (0)
+        if (nv <= 1)
+            ATX_QK_VEC_XT(1);
+        else if (nv == 2)
+            ATX_QK_VEC_XT(2);
+        else
+            ATX_QK_VEC_XT(4);
+#undef ATX_QK_VEC_XT
+#undef ATX_QK_VEC
+        return ATX_OK;
     }
     if (dtype == ATX_DT_F32) {
         if (smem > 48 * 1024)

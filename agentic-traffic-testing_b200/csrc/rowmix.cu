@@ -37,6 +37,22 @@ __device__ __forceinline__ void rst4(__nv_bfloat16* p, long long i4, float4 v) {
     reinterpret_cast<uint2*>(p)[i4] = make_uint2(pack_bf16(v.x, v.y), pack_bf16(v.z, v.w));
 }
 
+// Four elements as they are stored (bf16: two registers instead of four).
+template <typename XT>
+struct Raw4;
+template <>
+struct Raw4<float> {
+    float4 r;
+    __device__ __forceinline__ void load(const float* p, long long i4) { r = reinterpret_cast<const float4*>(p)[i4]; }
+    __device__ __forceinline__ float4 get() const { return r; }
+};
+template <>
+struct Raw4<__nv_bfloat16> {
+    uint2 r;
+    __device__ __forceinline__ void load(const __nv_bfloat16* p, long long i4) { r = reinterpret_cast<const uint2*>(p)[i4]; }
+    __device__ __forceinline__ float4 get() const { return make_float4(bf16lo(r.x), bf16hi(r.x), bf16lo(r.y), bf16hi(r.y)); }
+};
+
 static void set_pdl_row(cudaLaunchConfig_t& cfg, cudaLaunchAttribute* attr, int flags) {
     if (flags & ATX_FLAG_PDL) {
         attr[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
@@ -284,42 +300,63 @@ parallel_resid_norm_kernel(const __grid_constant__ ParallelResidArgs a) {
     const float sc = a.tm.y_scale;
     float ss = 0.f;
     if constexpr (NV > 0) {
+        // Every loop below issues its NV loads before anything uses or stores one of them.
         float4 v[NV];
-        if (tw) {
-            float s0 = 0.f;
-#pragma unroll
-            for (int n = 0; n < NV; ++n) {
-                const int i = threadIdx.x + n * blockDim.x;
-                if (i >= W4) continue;
-                const float4 e = rld4(er, i);
-                s0 += e.x * e.x + e.y * e.y + e.z * e.z + e.w * e.w;
-            }
-            rs0 = rsqrtf(row_sum(s0, red) / static_cast<float>(W) + a.eps);
-            __syncthreads();   // red is used again for the outgoing norm
-        }
+        Raw4<XT> ga[NV], gb[NV];
+        bool on[NV];
 #pragma unroll
         for (int n = 0; n < NV; ++n) {
             const int i = threadIdx.x + n * blockDim.x;
+            on[n] = i < W4;
             v[n] = make_float4(0.f, 0.f, 0.f, 0.f);
-            if (i >= W4) continue;
-            v[n] = start ? rld4(er, i) : rld4(hr, i);
-            if (tw) {
-                const float4 g = rld4(tw, i);
+            if (on[n]) v[n] = start ? rld4(er, i) : rld4(hr, i);
+        }
+        if (NV > 1) {   // the norm weights are on their way while the row is summed
+#pragma unroll
+            for (int n = 0; n < NV; ++n) {
+                const int i = threadIdx.x + n * blockDim.x;
+                if (wa && on[n]) ga[n].load(wa, i);
+                if (wb && on[n]) gb[n].load(wb, i);
+            }
+        }
+        if (tw) {
+            float s0 = 0.f;
+#pragma unroll
+            for (int n = 0; n < NV; ++n) s0 += v[n].x * v[n].x + v[n].y * v[n].y + v[n].z * v[n].z + v[n].w * v[n].w;
+            rs0 = rsqrtf(row_sum(s0, red) / static_cast<float>(W) + a.eps);
+            __syncthreads();   // red is used again for the outgoing norm
+#pragma unroll
+            for (int n = 0; n < NV; ++n) {
+                if (!on[n]) continue;
+                const float4 g = rld4(tw, threadIdx.x + n * blockDim.x);
                 v[n].x *= rs0 * g.x, v[n].y *= rs0 * g.y, v[n].z *= rs0 * g.z, v[n].w *= rs0 * g.w;
             }
-            float4 add = make_float4(0.f, 0.f, 0.f, 0.f);
-            if (yr) {
-                add = rld4(yr, i);
-                if (a.tm.zero_y) rst4(yr, i, make_float4(0.f, 0.f, 0.f, 0.f));
+        }
+        auto add_row = [&](const float* src, float w) {
+            float4 e[NV];
+#pragma unroll
+            for (int n = 0; n < NV; ++n)
+                e[n] = on[n] ? rld4(src, threadIdx.x + n * blockDim.x) : make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+            for (int n = 0; n < NV; ++n) {
+                v[n].x = fmaf(w, e[n].x, v[n].x), v[n].y = fmaf(w, e[n].y, v[n].y);
+                v[n].z = fmaf(w, e[n].z, v[n].z), v[n].w = fmaf(w, e[n].w, v[n].w);
             }
-            for (int k = 0; k < top; ++k) {
-                if (s_row[k] < 0) continue;
-                const float4 e = *reinterpret_cast<const float4*>(a.tm.experts + s_row[k] + 4 * i);
-                const float w = s_w[k];
-                add.x = fmaf(w, e.x, add.x), add.y = fmaf(w, e.y, add.y), add.z = fmaf(w, e.z, add.z), add.w = fmaf(w, e.w, add.w);
+        };
+        if (yr) {
+            add_row(yr, sc);
+            if (a.tm.zero_y) {
+#pragma unroll
+                for (int n = 0; n < NV; ++n)
+                    if (on[n]) rst4(yr, threadIdx.x + n * blockDim.x, make_float4(0.f, 0.f, 0.f, 0.f));
             }
-            v[n].x = fmaf(sc, add.x, v[n].x), v[n].y = fmaf(sc, add.y, v[n].y);
-            v[n].z = fmaf(sc, add.z, v[n].z), v[n].w = fmaf(sc, add.w, v[n].w);
+        }
+        for (int k = 0; k < top; ++k)
+            if (s_row[k] >= 0) add_row(a.tm.experts + s_row[k], sc * s_w[k]);
+#pragma unroll
+        for (int n = 0; n < NV; ++n) {
+            const int i = threadIdx.x + n * blockDim.x;
+            if (!on[n]) continue;
             if (enter) {
                 const float4 e = rld4(er, i);
                 v[n].x += e.x, v[n].y += e.y, v[n].z += e.z, v[n].w += e.w;
@@ -338,14 +375,14 @@ parallel_resid_norm_kernel(const __grid_constant__ ParallelResidArgs a) {
 #pragma unroll
         for (int n = 0; n < NV; ++n) {
             const int i = threadIdx.x + n * blockDim.x;
-            if (i >= W4) continue;
+            if (!on[n]) continue;
             const float4 u = make_float4(v[n].x * rs, v[n].y * rs, v[n].z * rs, v[n].w * rs);
             if (a.out_a) {
-                const float4 g = NV == 1 ? wa4 : rld4(wa, i);
+                const float4 g = NV == 1 ? wa4 : ga[n].get();
                 rst4(oa, i, make_float4(u.x * (sh + g.x), u.y * (sh + g.y), u.z * (sh + g.z), u.w * (sh + g.w)));
             }
             if (a.out_b) {
-                const float4 g = NV == 1 ? wb4 : rld4(wb, i);
+                const float4 g = NV == 1 ? wb4 : gb[n].get();
                 rst4(ob, i, make_float4(u.x * (sh + g.x), u.y * (sh + g.y), u.z * (sh + g.z), u.w * (sh + g.w)));
             }
         }
