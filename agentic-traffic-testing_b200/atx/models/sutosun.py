@@ -115,17 +115,21 @@ class Config:
         for i, l in enumerate(self.layers):
             if l.get("weights_of") is None:
                 continue
-            j = int(l["weights_of"])
-            if not 0 <= j < len(self.layers) or self.layers[j].get("weights_of") is not None:
-                raise ValueError(f"layer {i}: weights_of={j} must name a layer with tensors of its own")
+            j, seen = i, {i}
+            while self.layers[j].get("weights_of") is not None:
+                j = int(self.layers[j]["weights_of"])
+                if not 0 <= j < len(self.layers) or j in seen:
+                    raise ValueError(f"layer {i}: weights_of={l['weights_of']} must lead to a layer with tensors of its own")
+                seen.add(j)
             o = self.layers[j]
             if (o["type"], o["mixer"], o.get("mlp")) != (l["type"], l["mixer"], l.get("mlp")):
                 raise ValueError(f"layer {i}: uses layer {j}'s tensors but differs from it")
 
     def source(self, i: int) -> int:
         """The layer whose tensors layer i runs."""
-        j = self.layers[i].get("weights_of")
-        return i if j is None else int(j)
+        while self.layers[i].get("weights_of") is not None:
+            i = int(self.layers[i]["weights_of"])
+        return i
 
     @property
     def recurrent(self) -> bool:

@@ -58,6 +58,12 @@ def test_config_is_read_from_json_and_picked_by_architecture(tmp_path):
         d[path[-1]] = value
         with pytest.raises(ValueError):
             sutosun.Config.from_json(bad)
+    chain = json.loads(json.dumps(small_cfg(layers=cfg["layers"] + [dict(cfg["layers"][3], weights_of=3)])))      # through a layer that borrows itself
+    m5 = sutosun.Config.from_json(chain)
+    assert [m5.source(i) for i in range(5)] == [0, 1, 2, 1, 1] and m5.tensor_shapes() == m.tensor_shapes()
+    chain["layers"][3]["weights_of"] = 4
+    with pytest.raises(ValueError):
+        sutosun.Config.from_json(chain)
     plain = json.loads(json.dumps(cfg))           # what a configuration leaves out does not exist
     del plain["logit_softcap"], plain["layers"][0]["mixer"]["rot"]
     for l in (1, 3):
